@@ -22,7 +22,8 @@
 // (decoded tokens) all warps share the rows and each visits 16 of the 64 keys, keeping its own
 // (m, l, o); the four are merged through shared memory, in the order of the warps, at the end.
 //
-// Head sizes: any multiple of 8 up to 128 (padded with zeros to 64 or 128 in shared memory).
+// Head sizes: any multiple of 8 up to 128 (padded with zeros to 64 or 128 in shared memory), keys (and queries) and
+// values each their own.
 #include "common.cuh"
 
 #include <cuda.h>
@@ -38,7 +39,7 @@ constexpr int FA_THREADS = 128;
 
 struct FlashParams {
   const bf16* q; bf16* out;                 // [T, nq, d]
-  const bf16* k_cache; const bf16* v_cache; // [pages, nkv, page_size, d]
+  const bf16* k_cache; const bf16* v_cache; // [pages, nkv, page_size, d] (values: v_dim)
   const int* positions;                     // [T]
   const int* block_table; int max_pages;    // [S, max_pages]
   const int4* tiles;                        // {first token, tokens, request index, unused}
@@ -47,13 +48,15 @@ struct FlashParams {
   int part_rows;                            // most query rows of any tile
   int cluster;                              // > 0: the splits of a tile form a cluster of this size and combine through shared memory
   int num_q_heads, num_kv_heads, head_dim, group, page_size, page_shift, window, splits;   // page_shift: log2(page_size) or -1
+  int v_dim;                                // size of a value head: out is [T, nq, v_dim], the value pools' rows have v_dim
   float scale_log2;                         // scale * log2(e)
   int kv_share;                             // >= 1: the cache has num_kv_heads / kv_share heads, and kv head j of this launch
                                             // reads cache head j / kv_share (several groups of query heads on one cached head)
   const float* slopes;                      // optional [num_q_heads]: the score of key j for the query at position i is
   float inv_scale;                          // lowered by slopes[h] * (i - j); 1 / scale brings that into the raw score's units
+  float cap_raw, cap_exp;                   // cap_raw > 0: raw score s <- cap_raw * tanh(s / cap_raw), cap_raw = softcap / scale,
+                                            // cap_exp = 2 log2(e) / cap_raw
   // Three options of the kernel that fetches with 16-byte copies (the TMA kernel takes none of them):
-  float cap_raw, inv_cap_raw;               // cap_raw > 0: raw score s <- cap_raw * tanh(s * inv_cap_raw), cap_raw = softcap / scale
   const float* sinks;                       // optional [num_q_heads]: the denominator also holds exp(sinks[h]); needs scale > 0
   int pool;                                 // P > 0: behind the window a row at position i also sees entry b of a second paged
   const bf16* pool_k; const bf16* pool_v;   // cache (same page size and heads) for every b with (b + 1) P - 1 <= i - window,
@@ -119,7 +122,7 @@ template <int DP, bool NAMED>
 __device__ __forceinline__ void keysplit_finish(const FlashParams& p, float* scratch, float* fin, const float (&o)[DP / 8][4],
                                                 const float (&m_run)[2], const float (&l_run)[2], int t0, int rows, int kvh, int split) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int G = p.group, d = p.head_dim;
+  const int G = p.group, d = p.v_dim;
   // Merge the four warps' (m, l, o) through shared memory (the stages are no longer needed).
   keysplit_sync<NAMED>();
   constexpr int MS = DP + 8;
@@ -207,14 +210,18 @@ __device__ __forceinline__ void keysplit_finish(const FlashParams& p, float* scr
   }
 }
 
-template <int DP, bool KEYSPLIT>
+// DP, DV: padded sizes of a key and of a value head
+template <int DP, int DV, bool KEYSPLIT>
 __global__ void __launch_bounds__(FA_THREADS, KEYSPLIT ? 2 : 3)
 flash_attention_kernel(FlashParams p) {
   constexpr int CHUNKS = DP / 8;                  // 16-byte chunks of a row
+  constexpr int V_CHUNKS = DV / 8;
   constexpr int NB = KEYSPLIT ? 2 : FA_KEYS / 8;  // blocks of 8 keys a warp visits in a stage
   constexpr int LOADS = FA_KEYS * CHUNKS / FA_THREADS;      // 16-byte copies a thread makes per stage and matrix
+  constexpr int V_LOADS = FA_KEYS * V_CHUNKS / FA_THREADS;
   constexpr int ROW_STEP = FA_THREADS / CHUNKS;             // rows between two copies of one thread
-  constexpr int TILE_BYTES = FA_KEYS * DP * 2;
+  constexpr int V_ROW_STEP = FA_THREADS / V_CHUNKS;
+  constexpr int TILE_BYTES = FA_KEYS * DP * 2, V_TILE_BYTES = FA_KEYS * DV * 2;
   // Decoded tokens: three stages, bound by memory.  Portions of prompts: two stages, and the query tile
   // lies on the second stage's keys (it is in registers before that stage is first filled), so that a CTA
   // needs 64 KB and three of them share an SM.
@@ -230,7 +237,7 @@ flash_attention_kernel(FlashParams p) {
   const int4 tile = p.tiles[blockIdx.x];
   const int t0 = tile.x, ntok = tile.y, seq = tile.z;
   const int kvh = blockIdx.y, split = blockIdx.z;
-  const int G = p.group, d = p.head_dim;
+  const int G = p.group, d = p.head_dim, dv = p.v_dim;
   const int rows = ntok * G;
   const int pos0 = p.positions[t0];
   const int pos_last = pos0 + ntok - 1;
@@ -279,11 +286,18 @@ flash_attention_kernel(FlashParams p) {
   const uint32_t ld_smem = tile_offset<DP>(ld_row, ld_chunk);
   const size_t head_off = (size_t)(kvh / p.kv_share) * p.page_size * d + ld_chunk * 8;
   const size_t page_stride = (size_t)(p.num_kv_heads / p.kv_share) * p.page_size * d;
+  // the values' columns, where their size differs (with one size the two sets of copies share all of this)
+  const bool one_size = d == dv;
+  const int v_row = tid / V_CHUNKS, v_chunk = tid % V_CHUNKS;
+  const bool v_col_valid = v_chunk * 8 < dv;
+  const uint32_t v_ld_smem = tile_offset<DV>(v_row, v_chunk);
+  const size_t v_head_off = (size_t)(kvh / p.kv_share) * p.page_size * dv + v_chunk * 8;
+  const size_t v_page_stride = (size_t)(p.num_kv_heads / p.kv_share) * p.page_size * dv;
   auto load_stage = [&](int stage_idx) {
     const int buf = stage_idx % STAGES;
     const int u0 = ubeg + stage_idx * FA_KEYS;
     const bool pooled = u0 < PB;                 // a stage of pooled entries: the second cache through its own table
-    const int kbase = (pooled ? u0 : lo_tile + (u0 - PB)) + ld_row;
+    const int kfirst = pooled ? u0 : lo_tile + (u0 - PB), kbase = kfirst + ld_row;
     const int end = pooled ? eend : kend;
     const int* tbl = pooled ? pool_bt : bt;
     const bf16* kc = pooled ? p.pool_k : p.k_cache;
@@ -294,15 +308,39 @@ flash_attention_kernel(FlashParams p) {
       const int j = kbase + i * ROW_STEP;
       const int pi = p.page_shift >= 0 ? (j >> p.page_shift) : (j / p.page_size);
       slot[i] = j - pi * p.page_size;
-      page[i] = (j < end && ld_col_valid) ? tbl[pi] : -1;
+      page[i] = (j < end && (ld_col_valid || (DP == DV && v_col_valid))) ? tbl[pi] : -1;
     }
 #pragma unroll
     for (int i = 0; i < LOADS; ++i) {
-      const bool valid = page[i] >= 0;
+      const bool valid = page[i] >= 0 && ld_col_valid;
       const size_t off = valid ? (size_t)page[i] * page_stride + head_off + (size_t)slot[i] * d : 0;
       const uint32_t so = buf * TILE_BYTES + ld_smem + i * ROW_STEP * (DP * 2);
       cp_async16(k_smem + so, kc + off, valid);
-      cp_async16(v_smem + so, vc + off, valid);
+      if (DP == DV) {                            // one padded size: the same rows and columns, though the sizes may differ
+        if (one_size) {
+          cp_async16(v_smem + so, vc + off, valid);
+        } else {
+          const bool vv = page[i] >= 0 && v_col_valid;
+          cp_async16(v_smem + so, vc + (vv ? (size_t)page[i] * v_page_stride + v_head_off + (size_t)slot[i] * dv : 0), vv);
+        }
+      }
+    }
+    if (DP != DV) {
+      const int vbase = kfirst + v_row;
+      int vpage[V_LOADS], vslot[V_LOADS];
+#pragma unroll
+      for (int i = 0; i < V_LOADS; ++i) {
+        const int j = vbase + i * V_ROW_STEP;
+        const int pi = p.page_shift >= 0 ? (j >> p.page_shift) : (j / p.page_size);
+        vslot[i] = j - pi * p.page_size;
+        vpage[i] = (j < end && v_col_valid) ? tbl[pi] : -1;
+      }
+#pragma unroll
+      for (int i = 0; i < V_LOADS; ++i) {
+        const bool vv = vpage[i] >= 0;
+        cp_async16(v_smem + buf * V_TILE_BYTES + v_ld_smem + i * V_ROW_STEP * (DV * 2),
+                   vc + (vv ? (size_t)vpage[i] * v_page_stride + v_head_off + (size_t)vslot[i] * dv : 0), vv);
+      }
     }
   };
 
@@ -340,9 +378,9 @@ flash_attention_kernel(FlashParams p) {
     }
   }
 
-  float o[DP / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < DP / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 
   for (int st = 0; st < num_stages; ++st) {
@@ -353,7 +391,7 @@ flash_attention_kernel(FlashParams p) {
     if (!warp_active) continue;
 
     const int buf = st % STAGES;
-    const uint32_t kb = k_smem + buf * TILE_BYTES, vb = v_smem + buf * TILE_BYTES;
+    const uint32_t kb = k_smem + buf * TILE_BYTES, vb = v_smem + buf * V_TILE_BYTES;
     const int u0 = ubeg + st * FA_KEYS;
     const bool pooled = u0 < PB;
     const int kbase = pooled ? u0 : lo_tile + (u0 - PB);      // the stage's first pooled entry or key
@@ -388,10 +426,7 @@ flash_attention_kernel(FlashParams p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int h = e >> 1;
-        if (p.cap_raw > 0.f) {                              // tanh(x) = 1 - 2 / (exp(2 x) + 1), exact at both ends
-          const float ex = __expf(2.f * s[nb][e] * p.inv_cap_raw);
-          s[nb][e] = p.cap_raw * (1.f - __fdividef(2.f, ex + 1.f));
-        }
+        if (p.cap_raw > 0.f) s[nb][e] = capped_score(s[nb][e], p.cap_raw, p.cap_exp);
         if (need_mask || biased) {
           const int j = kbase + key0 + nb * 8 + (lane & 3) * 2 + (e & 1);
           if (biased) s[nb][e] = fmaf(-row_bias[h], (float)(row_pos[h] - j), s[nb][e]);
@@ -429,7 +464,7 @@ flash_attention_kernel(FlashParams p) {
     // Once the maxima have settled the factors are exactly 1 for stage after stage: skip the multiplications then.
     if (!__all_sync(0xffffffffu, alpha[0] == 1.f && alpha[1] == 1.f)) {
 #pragma unroll
-      for (int i = 0; i < DP / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         o[i][0] *= alpha[0]; o[i][1] *= alpha[0]; o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
       }
     }
@@ -438,12 +473,12 @@ flash_attention_kernel(FlashParams p) {
 #pragma unroll
     for (int ks = 0; ks < NB / 2; ++ks) {
 #pragma unroll
-      for (int db = 0; db < DP / 8; db += 2) {
+      for (int db = 0; db < DV / 8; db += 2) {
         // matrices (transposed on load): (keys lo, dims db), (keys hi, dims db), (keys lo, dims db+1), (keys hi, dims db+1)
         const int key = key0 + ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
         const int c = db + (lane >> 4);
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(vb + tile_offset<DP>(key, c), b0, b1, b2, b3);
+        ldmatrix_x4_trans(vb + tile_offset<DV>(key, c), b0, b1, b2, b3);
         mma_bf16(o[db], pf[ks], b0, b1);
         mma_bf16(o[db + 1], pf[ks], b2, b3);
       }
@@ -462,7 +497,7 @@ flash_attention_kernel(FlashParams p) {
       const float a = m_run[h] == -INFINITY ? 0.f : exp2f((m_run[h] - m_new) * p.scale_log2);
       l_run[h] = l_run[h] * a + ((lane & 3) == 0 ? exp2f((sink - m_new) * p.scale_log2) : 0.f);
 #pragma unroll
-      for (int i = 0; i < DP / 8; ++i) { o[i][2 * h] *= a; o[i][2 * h + 1] *= a; }
+      for (int i = 0; i < DV / 8; ++i) { o[i][2 * h] *= a; o[i][2 * h + 1] *= a; }
       m_run[h] = m_new;
     }
   }
@@ -474,8 +509,9 @@ flash_attention_kernel(FlashParams p) {
     l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
   }
   if (KEYSPLIT) {
-    keysplit_finish<DP, false>(p, reinterpret_cast<float*>(smem + FA_ROWS * DP * 2),
-                               reinterpret_cast<float*>(smem + FA_ROWS * DP * 2 + STAGES * TILE_BYTES), o, m_run, l_run, t0, rows, kvh, split);
+    float* scratch = reinterpret_cast<float*>(smem + Q_BYTES);               // the stages, keys' and values', are free by now
+    static_assert((keysplit_scratch_floats(DV) + 16 * (DV + 2)) * 4 <= FA_STAGES * (TILE_BYTES + V_TILE_BYTES), "the merge fits the stages");
+    keysplit_finish<DV, false>(p, scratch, scratch + keysplit_scratch_floats(DV), o, m_run, l_run, t0, rows, kvh, split);
     return;
   }
   if (!warp_active) return;
@@ -486,19 +522,19 @@ flash_attention_kernel(FlashParams p) {
     const int token = t0 + r / G, head = kvh * G + r % G;
     if (p.splits == 1) {
       const float inv = l_run[h] > 0.f ? 1.f / l_run[h] : 0.f;
-      bf16* dst = p.out + ((size_t)token * p.num_q_heads + head) * d;
+      bf16* dst = p.out + ((size_t)token * p.num_q_heads + head) * dv;
 #pragma unroll
-      for (int i = 0; i < DP / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         const int dim = i * 8 + (lane & 3) * 2;
-        if (dim < d) *reinterpret_cast<__nv_bfloat162*>(dst + dim) = __floats2bfloat162_rn(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
+        if (dim < dv) *reinterpret_cast<__nv_bfloat162*>(dst + dim) = __floats2bfloat162_rn(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
       }
     } else {
       const size_t slot = (((size_t)blockIdx.x * p.num_kv_heads + kvh) * p.splits + split) * p.part_rows + r;
-      float* dst = p.part_o + slot * d;
+      float* dst = p.part_o + slot * dv;
 #pragma unroll
-      for (int i = 0; i < DP / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         const int dim = i * 8 + (lane & 3) * 2;
-        if (dim < d) *reinterpret_cast<float2*>(dst + dim) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
+        if (dim < dv) *reinterpret_cast<float2*>(dst + dim) = make_float2(o[i][2 * h], o[i][2 * h + 1]);
       }
       if ((lane & 3) == 0) {
         p.part_ml[slot * 2 + 0] = m_run[h] == -INFINITY ? -INFINITY : m_run[h] * p.scale_log2;
@@ -566,13 +602,14 @@ __device__ __forceinline__ uint32_t fd_offset(int key, int chunk) {
   return (uint32_t)((chunk >> 3) * 8192 + key * 128 + (((chunk & 7) ^ (key & 7)) << 4));
 }
 
-template <int DP>
+template <int DP, int DV>
 __global__ void __launch_bounds__(FD_THREADS, 2)
 flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap, FlashParams p) {
   constexpr int CHUNKS = DP / 8;
-  constexpr int NH = DP / 64;                       // halves of 64 dimensions
-  constexpr int MAT_BYTES = NH * 8192;              // a stage's keys (or values)
-  constexpr int STAGE_BYTES = 2 * MAT_BYTES;
+  constexpr int V_CHUNKS = DV / 8;
+  constexpr int NH = DP / 64, NHV = DV / 64;        // halves of 64 dimensions, of keys and of values
+  constexpr int MAT_BYTES = NH * 8192;              // a stage's keys
+  constexpr int STAGE_BYTES = MAT_BYTES + NHV * 8192;
   extern __shared__ uint8_t fd_smem_raw[];
   __shared__ __align__(8) unsigned long long bars[2 * FD_STAGES];
   __shared__ int abort_word;
@@ -611,10 +648,11 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
   __syncthreads();
 
   if (warp == 4) {
-    // ---- the fetching warp: lane = (box of keys, half of the dimensions, keys or values) ----------------------------------
+    // ---- the fetching warp: lane = (box of keys, half of the keys' or of the values' dimensions) --------------------------
     const int box_keys = min(p.page_size, FA_KEYS);
-    const int nops = 2 * NH * (FA_KEYS / box_keys);
-    const int kv = lane & 1, half = (lane >> 1) % NH, box = (lane >> 1) / NH;
+    const int nops = (NH + NHV) * (FA_KEYS / box_keys);
+    const int which = lane % (NH + NHV), box = lane / (NH + NHV);
+    const int kv = which >= NH ? 1 : 0, half = kv ? which - NH : which;
     const bool active = lane < nops;
     const CUtensorMap* map = kv ? &vmap : &kmap;
     const uint32_t dst_off = (uint32_t)(kv * MAT_BYTES + half * 8192 + box * box_keys * 128);
@@ -677,9 +715,9 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
     ldmatrix_x4(q_smem + tile_offset<DP>(r, c), qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
   }
 
-  float o[DP / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < DP / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int key0 = warp * 16;                        // the 16 keys of a stage this warp visits
 
@@ -708,8 +746,8 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
     // times a NaN is not).
     if (kbase + FA_KEYS > kend || kbase < lo_tile) {
       const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-      for (int idx = lane; idx < 16 * CHUNKS; idx += 32) {
-        const int key = key0 + idx / CHUNKS, c = idx % CHUNKS;
+      for (int idx = lane; idx < 16 * V_CHUNKS; idx += 32) {
+        const int key = key0 + idx / V_CHUNKS, c = idx % V_CHUNKS;
         if (kbase + key >= kend || kbase + key < lo_tile)
           *reinterpret_cast<uint4*>(base_ptr + b * STAGE_BYTES + MAT_BYTES + fd_offset(key, c)) = zero;
       }
@@ -725,6 +763,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int h = e >> 1;
+        if (p.cap_raw > 0.f) s[nb][e] = capped_score(s[nb][e], p.cap_raw, p.cap_exp);
         if (need_mask || p.slopes) {
           const int j = kbase + key0 + nb * 8 + (lane & 3) * 2 + (e & 1);
           s[nb][e] = fmaf(-row_bias[h], (float)(row_pos[h] - j), s[nb][e]);
@@ -760,14 +799,14 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
     for (int h = 0; h < 2; ++h) l_run[h] = l_run[h] * alpha[h] + row_sum[h];
     if (!__all_sync(0xffffffffu, alpha[0] == 1.f && alpha[1] == 1.f)) {
 #pragma unroll
-      for (int i = 0; i < DP / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         o[i][0] *= alpha[0]; o[i][1] *= alpha[0]; o[i][2] *= alpha[1]; o[i][3] *= alpha[1];
       }
     }
 
     // ---- O += P V ------------------------------------------------------------------------------------------------------------
 #pragma unroll
-    for (int db = 0; db < DP / 8; db += 2) {
+    for (int db = 0; db < DV / 8; db += 2) {
       // matrices (transposed on load): (keys lo, dims db), (keys hi, dims db), (keys lo, dims db+1), (keys hi, dims db+1)
       const int key = key0 + (lane & 7) + ((lane >> 3) & 1) * 8;
       const int c = db + (lane >> 4);
@@ -787,7 +826,8 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
   }
   // the stages are free now (every copy that was issued has been waited for): the merge uses them
   float* scratch = reinterpret_cast<float*>(base_ptr);
-  keysplit_finish<DP, true>(p, scratch, scratch + keysplit_scratch_floats(DP), o, m_run, l_run, t0, rows, kvh, split);
+  static_assert((keysplit_scratch_floats(DV) + 16 * (DV + 2)) * 4 <= FD_STAGES * STAGE_BYTES, "the merge fits the stages");
+  keysplit_finish<DV, true>(p, scratch, scratch + keysplit_scratch_floats(DV), o, m_run, l_run, t0, rows, kvh, split);
 }
 
 // Combines the partials of the splits, in their order: out = sum_z o_z 2^(m_z - M) / sum_z l_z 2^(m_z - M).
@@ -802,7 +842,7 @@ __global__ void flash_combine_kernel(FlashParams p) {
   pdl_wait();
   const int4 tile = p.tiles[blockIdx.x];
   const int kvh = blockIdx.y;
-  const int rows = tile.y * p.group, d = p.head_dim;
+  const int rows = tile.y * p.group, d = p.v_dim;
   const int lane = threadIdx.x, warp = threadIdx.y, nwarps = blockDim.y;
   float* wz = wsm + warp * p.splits;
   const size_t base = ((size_t)blockIdx.x * p.num_kv_heads + kvh) * p.splits;
@@ -919,7 +959,7 @@ LB_EXPORT int lb_attention_flash_wide_clusters(int head_dim) {
   const int dp = head_dim <= 64 ? 64 : 128;
   int& c = cached[dp == 64];
   if (c >= 0) return c;
-  void (*kern)(CUtensorMap, CUtensorMap, lb::FlashParams) = dp == 64 ? lb::flash_decode_tma_kernel<64> : lb::flash_decode_tma_kernel<128>;
+  void (*kern)(CUtensorMap, CUtensorMap, lb::FlashParams) = dp == 64 ? lb::flash_decode_tma_kernel<64, 64> : lb::flash_decode_tma_kernel<128, 128>;
   const int fd_smem = 1024 + lb::FD_STAGES * 2 * (dp / 64) * 8192 + 16 * dp * 2;
   c = 0;
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess ||
@@ -939,7 +979,7 @@ LB_EXPORT int lb_attention_flash_wide_clusters(int head_dim) {
   return c;
 }
 
-// Floats of workspace a launch with these sizes needs (partials of o, then of m and l).
+// Floats of workspace a launch with these sizes needs (partials of o, then of m and l); head_dim: the values'.
 LB_EXPORT long long lb_attention_flash_workspace(int num_tiles, int num_kv_heads, int splits, int part_rows, int head_dim) {
   if (splits <= 1) return 0;
   return (long long)num_tiles * num_kv_heads * splits * part_rows * (head_dim + 2);
@@ -954,14 +994,16 @@ LB_EXPORT long long lb_attention_flash_workspace(int num_tiles, int num_kv_heads
 // denominator also holds exp(sinks[h]).  pool = P > 0 (needs a window): a query at position i also sees entry b of the
 // second paged cache pool_k / pool_v (same page size and heads, block table pool_table with pool_max_pages columns) for
 // every b with (b + 1) P - 1 <= i - window.  chunk = C > 0: positions in runs of C from the sequence's start, a query sees
-// its own run only.  Any of the four keeps the launch off the TMA kernel.
+// its own run only.  Sinks, pooled blocks and chunks keep the launch off the TMA kernel.  v_dim: the size of a value
+// head if it is not head_dim (0: it is); out is then [T, nq, v_dim].
 LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cache, const void* v_cache,
                                     const int* positions, const int* block_table, const void* tiles, int num_tiles,
                                     int num_q_heads, int num_kv_heads, int head_dim, int page_size, int max_pages,
                                     int num_pages, int window, float scale, int splits, int part_rows, float* workspace,
                                     long long workspace_elems, int kv_share, const float* slopes, float softcap,
                                     const float* sinks, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
-                                    int pool_max_pages, int chunk, cudaStream_t stream) {
+                                    int pool_max_pages, int chunk, int v_dim, cudaStream_t stream) {
+  if (v_dim <= 0) v_dim = head_dim;
   LB_CHECK_ARG(chunk >= 0 && (chunk == 0 || pool == 0), "attention_flash: chunks of %d keys (and no pooled blocks with them)", chunk);
   LB_CHECK_ARG((slopes == nullptr && sinks == nullptr && !(softcap > 0.f)) || scale > 0.f,
                "attention_flash: a distance bias, a cap and a sink need a positive scale");
@@ -969,7 +1011,7 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
   LB_CHECK_ARG(pool == 0 || (pool > 0 && window > 0 && pool_k && pool_v && pool_table && pool_max_pages > 0 && kv_share == 1 &&
                              ((uintptr_t)pool_k % 16 == 0) && ((uintptr_t)pool_v % 16 == 0)),
                "attention_flash: pooled blocks need a window, the pooled cache and its block table");
-  if (softcap > 0.f || sinks || pool > 0 || chunk > 0) num_pages = 0;
+  if (sinks || pool > 0 || chunk > 0) num_pages = 0;
   LB_CHECK_ARG(num_q_heads > 0 && num_kv_heads > 0 && num_q_heads % num_kv_heads == 0,
                "attention_flash: %d query heads are not a multiple of %d kv heads", num_q_heads, num_kv_heads);
   LB_CHECK_ARG(kv_share >= 1 && num_kv_heads % kv_share == 0, "attention_flash: %d kv heads cannot share cached heads %d by %d",
@@ -978,6 +1020,7 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
   LB_CHECK_ARG(group <= lb::FA_ROWS, "attention_flash: %d query heads per kv head, at most %d", group, lb::FA_ROWS);
   LB_CHECK_ARG(head_dim >= 8 && head_dim <= 128 && head_dim % 8 == 0,
                "attention_flash: head_dim %d must be a multiple of 8 between 8 and 128", head_dim);
+  LB_CHECK_ARG(v_dim >= 8 && v_dim <= 128 && v_dim % 8 == 0, "attention_flash: value size %d must be a multiple of 8 between 8 and 128", v_dim);
   const bool force_workspace = splits < 0;     // a negative count asks for the path through the workspace
   if (splits < 0) splits = -splits;
   LB_CHECK_ARG(page_size > 0 && max_pages > 0 && window >= 0 && splits >= 1 && splits <= 65535, "attention_flash: bad sizes");
@@ -993,27 +1036,27 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
   // Up to 8 splits (a power of two) of tiles of at most 16 rows combine inside a thread-block cluster; the TMA kernel
   // also takes clusters of 16 (a size the launch has to ask for: not every GPU schedules it).
   const bool may_cluster = part_rows <= 16 && splits <= (by_tma ? 16 : 8) && !force_workspace;
-  LB_CHECK_ARG(splits == 1 || may_cluster || (workspace && workspace_elems >= lb_attention_flash_workspace(num_tiles, num_kv_heads, splits, part_rows, head_dim)),
+  LB_CHECK_ARG(splits == 1 || may_cluster || (workspace && workspace_elems >= lb_attention_flash_workspace(num_tiles, num_kv_heads, splits, part_rows, v_dim)),
                "attention_flash: the workspace is too small for %d splits", splits);
   lb::FlashParams p;
   p.q = (const lb::bf16*)q; p.out = (lb::bf16*)out; p.k_cache = (const lb::bf16*)k_cache; p.v_cache = (const lb::bf16*)v_cache;
   p.positions = positions; p.block_table = block_table; p.max_pages = max_pages; p.tiles = (const int4*)tiles;
   p.part_o = workspace;
-  p.part_ml = workspace ? workspace + (long long)num_tiles * num_kv_heads * splits * part_rows * head_dim : nullptr;
+  p.part_ml = workspace ? workspace + (long long)num_tiles * num_kv_heads * splits * part_rows * v_dim : nullptr;
   p.part_rows = part_rows;
   p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.head_dim = head_dim; p.group = group;
-  p.page_size = page_size; p.window = window; p.splits = splits;
+  p.page_size = page_size; p.window = window; p.splits = splits; p.v_dim = v_dim;
   p.page_shift = page_shift;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.kv_share = kv_share;
   p.slopes = slopes; p.inv_scale = (slopes || sinks) ? 1.f / scale : 0.f;
-  p.cap_raw = softcap > 0.f ? softcap / scale : 0.f; p.inv_cap_raw = softcap > 0.f ? scale / softcap : 0.f;
+  p.cap_raw = softcap > 0.f ? softcap / scale : 0.f; p.cap_exp = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   p.sinks = sinks; p.pool = pool; p.pool_k = (const lb::bf16*)pool_k; p.pool_v = (const lb::bf16*)pool_v;
   p.pool_table = pool_table; p.pool_max_pages = pool_max_pages; p.chunk = chunk;
   dim3 grid(num_tiles, num_kv_heads, splits);
-  const int dp = head_dim <= 64 ? 64 : 128;
-  const int smem = part_rows <= 16 ? (lb::FA_ROWS + 2 * lb::FA_STAGES * lb::FA_KEYS) * dp * 2   // query tile + 3 stages
-                                   : 2 * 2 * lb::FA_KEYS * dp * 2;                             // 2 stages, query tile aliased
+  const int dp = head_dim <= 64 ? 64 : 128, dpv = v_dim <= 64 ? 64 : 128;
+  const int smem = part_rows <= 16 ? lb::FA_ROWS * dp * 2 + lb::FA_STAGES * lb::FA_KEYS * (dp + dpv) * 2   // query tile + 3 stages
+                                   : 2 * lb::FA_KEYS * (dp + dpv) * 2;                                    // 2 stages, query tile aliased
   const bool keysplit = part_rows <= 16;      // no tile has more than 16 query rows: the warps share them
   const bool clustered = splits > 1 && may_cluster;
   p.cluster = clustered ? splits : 0;
@@ -1021,18 +1064,20 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
     CUtensorMap mk, mv;
     const long long pool_rows = (long long)num_pages * (num_kv_heads / kv_share) * page_size;
     const int box = page_size < lb::FA_KEYS ? page_size : lb::FA_KEYS;
-    if (!lb::fd_pool_map(&mk, k_cache, pool_rows, head_dim, box) || !lb::fd_pool_map(&mv, v_cache, pool_rows, head_dim, box)) {
+    if (!lb::fd_pool_map(&mk, k_cache, pool_rows, head_dim, box) || !lb::fd_pool_map(&mv, v_cache, pool_rows, v_dim, box)) {
       lb::set_error("attention_flash: cuTensorMapEncodeTiled failed (pool of %lld rows of %d)", pool_rows, head_dim);
       return 3;
     }
-    const int fd_smem = 1024 + lb::FD_STAGES * 2 * (dp / 64) * 8192 + 16 * dp * 2;
-    static bool fd_cfg[2] = {false, false};
-    void (*kern)(CUtensorMap, CUtensorMap, lb::FlashParams) = dp == 64 ? lb::flash_decode_tma_kernel<64> : lb::flash_decode_tma_kernel<128>;
-    if (!fd_cfg[dp == 64]) {
+    const int fd_smem = 1024 + lb::FD_STAGES * ((dp + dpv) / 64) * 8192 + 16 * dp * 2;
+    static bool fd_cfg[4] = {false, false, false, false};
+    bool& fd_set = fd_cfg[(dp == 64) * 2 + (dpv == 64)];
+    void (*kern)(CUtensorMap, CUtensorMap, lb::FlashParams) = dp == 64 ? (dpv == 64 ? lb::flash_decode_tma_kernel<64, 64> : lb::flash_decode_tma_kernel<64, 128>)
+                                                                       : (dpv == 64 ? lb::flash_decode_tma_kernel<128, 64> : lb::flash_decode_tma_kernel<128, 128>);
+    if (!fd_set) {
       cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, fd_smem);
       if (e != cudaSuccess) { lb::set_error("attention_flash: cannot reserve %d bytes of shared memory: %s", fd_smem, cudaGetErrorString(e)); return 2; }
-      fd_cfg[dp == 64] = true;
+      fd_set = true;
     }
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid; cfg.blockDim = dim3(lb::FD_THREADS); cfg.dynamicSmemBytes = fd_smem; cfg.stream = stream;
@@ -1058,11 +1103,11 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
     }
     return 0;
   }
-#define LB_FLASH_LAUNCH(DP, KS)                                                                                 \
+#define LB_FLASH_LAUNCH(DP, DV, KS)                                                                                 \
   do {                                                                                                          \
     static bool cfg = false;                                                                                    \
     if (!cfg) {                                                                                                 \
-      cudaFuncSetAttribute(lb::flash_attention_kernel<DP, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
+      cudaFuncSetAttribute(lb::flash_attention_kernel<DP, DV, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); \
       cfg = true;                                                                                               \
     }                                                                                                           \
     if (clustered) {                                                                                            \
@@ -1074,13 +1119,18 @@ LB_EXPORT int lb_attention_flash_ex(const void* q, void* out, const void* k_cach
       attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;                                          \
       attr[1].val.programmaticStreamSerializationAllowed = 1;                                                   \
       cfg.attrs = attr; cfg.numAttrs = lb::g_pdl_enabled ? 2 : 1;                                               \
-      cudaLaunchKernelEx(&cfg, lb::flash_attention_kernel<DP, KS>, p);                                          \
+      cudaLaunchKernelEx(&cfg, lb::flash_attention_kernel<DP, DV, KS>, p);                                          \
     } else {                                                                                                    \
-      lb::launch(lb::flash_attention_kernel<DP, KS>, grid, dim3(lb::FA_THREADS), smem, stream, p);              \
+      lb::launch(lb::flash_attention_kernel<DP, DV, KS>, grid, dim3(lb::FA_THREADS), smem, stream, p);              \
     }                                                                                                           \
   } while (0)
-  if (dp == 64) { if (keysplit) LB_FLASH_LAUNCH(64, true); else LB_FLASH_LAUNCH(64, false); }
-  else { if (keysplit) LB_FLASH_LAUNCH(128, true); else LB_FLASH_LAUNCH(128, false); }
+#define LB_FLASH_SIZES(KS)                                                                      \
+  do {                                                                                          \
+    if (dp == 64) { if (dpv == 64) LB_FLASH_LAUNCH(64, 64, KS); else LB_FLASH_LAUNCH(64, 128, KS); } \
+    else { if (dpv == 64) LB_FLASH_LAUNCH(128, 64, KS); else LB_FLASH_LAUNCH(128, 128, KS); }        \
+  } while (0)
+  if (keysplit) LB_FLASH_SIZES(true); else LB_FLASH_SIZES(false);
+#undef LB_FLASH_SIZES
 #undef LB_FLASH_LAUNCH
   LB_CHECK_LAUNCH("attention_flash");
   if (splits > 1 && !clustered) {
@@ -1098,5 +1148,5 @@ LB_EXPORT int lb_attention_flash(const void* q, void* out, const void* k_cache, 
                                  long long workspace_elems, int kv_share, const float* slopes, cudaStream_t stream) {
   return lb_attention_flash_ex(q, out, k_cache, v_cache, positions, block_table, tiles, num_tiles, num_q_heads, num_kv_heads,
                                head_dim, page_size, max_pages, num_pages, window, scale, splits, part_rows, workspace,
-                               workspace_elems, kv_share, slopes, 0.f, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, stream);
+                               workspace_elems, kv_share, slopes, 0.f, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, 0, stream);
 }

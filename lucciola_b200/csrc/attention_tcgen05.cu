@@ -67,6 +67,8 @@ struct TcAttnParams {
   const int4* tiles;                        // {first token, tokens, request index, unused}
   int num_q_heads, num_kv_heads, group, page_size, page_shift, window;
   float scale_log2;
+  float cap_raw, cap_exp;                   // cap_raw > 0: raw score s <- cap_raw * tanh(s / cap_raw), cap_raw = softcap / scale,
+                                            // cap_exp = 2 log2(e) / cap_raw
   const float* slopes;                      // optional [num_q_heads]: the score of key j for the query at position i is lowered by
   float inv_scale;                          // slopes[h] * (i - j); 1 / scale brings that into the raw score's units
   // With gridDim.z > 1 the keys of every work item are cut into gridDim.z ranges of whole blocks, one CTA each; a CTA
@@ -445,6 +447,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
 #pragma unroll
         for (int j = 0; j < 64; ++j) x[j] = __uint_as_float(v[j]);
       }
+      if (p.cap_raw > 0.f) {
+#pragma unroll
+        for (int j = 0; j < TA_KEYS; ++j) x[j] = capped_score(x[j], p.cap_raw, p.cap_exp);
+      }
       if (p.slopes) {                                         // the distance bias, before the maximum is taken
         const float d0 = (float)(row_pos - kb);
 #pragma unroll
@@ -679,7 +685,8 @@ LB_EXPORT int lb_attention_tcgen05(const void* q, void* out, const void* k_cache
                                    const int* block_table, const void* tiles, int num_tiles, int num_tokens,
                                    int num_q_heads, int num_kv_heads, int head_dim, int page_size, int num_pages,
                                    int max_pages, int window, float scale, int key_splits, float* workspace,
-                                   long long workspace_elems, const float* slopes, cudaStream_t stream) {
+                                   long long workspace_elems, const float* slopes, float softcap, cudaStream_t stream) {
+  LB_CHECK_ARG(softcap >= 0.f && (softcap == 0.f || scale > 0.f), "attention_tcgen05: a cap of %f needs a positive scale", (double)softcap);
   LB_CHECK_ARG(slopes == nullptr || scale > 0.f, "attention_tcgen05: a distance bias needs a positive scale");
   LB_CHECK_ARG(lb_attention_tcgen05_ok(num_q_heads, num_kv_heads, head_dim, page_size),
                "attention_tcgen05: needs head_dim 128, at most 128 query heads per kv head and a page size among 8, 16, 32, 64, 128 "
@@ -708,6 +715,7 @@ LB_EXPORT int lb_attention_tcgen05(const void* q, void* out, const void* k_cache
   p.tiles = (const int4*)tiles; p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.group = group;
   p.page_size = page_size; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
   p.slopes = slopes; p.inv_scale = slopes ? 1.f / scale : 0.f;
+  p.cap_raw = softcap > 0.f ? softcap / scale : 0.f; p.cap_exp = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   p.page_shift = 0;
   while ((1 << p.page_shift) < page_size) ++p.page_shift;
   const int smem = lb::TA_SMEM_BYTES + 1024;

@@ -8,16 +8,18 @@
 //              by their sum + 1e-20, times `scale`.
 //   dispatch   the (token, choice) pairs sorted by expert: offsets of the experts' runs, the pair at each place and
 //              the place of each pair, and the list of row tiles (expert, first place) the products walk.  One CTA;
-//              nothing comes back to the host, so a step's launches do not depend on the choices.
+//              nothing comes back to the host, so a step's launches do not depend on the choices.  The experts of a pair are
+//              ids[pair], or, for models that choose by the token's id alone, table[token id, choice] with a table of the
+//              vocabulary's size: then there is no router and nothing of the step comes before this kernel.
 //   product    y[place, :] = act(x[row(place), :] . W[e]^T) for the places of expert e, W [experts, N, K].  With
 //              `gated`, W[e] holds N/2 gate rows and then N/2 up rows and y has N/2 columns (the activations of
-//              swiglu.cu).  row(place) is the pair's token for the first product (`gather`), the place itself for the second.
+//              swiglu.cu); without it, an element operation of post_op.cuh may follow the sum.  row(place) is the pair's token for the first product (`gather`), the place itself for the second.
 //   combine    out[t, :] = sum_k weight[t, k] * y[place(t, k), :] (+ an expert every token uses), k in the order
 //              of the choice, in 32-bit.
 //
 // Every output element is one thread's sum over k in increasing order, so a token's result does not depend on where
 // the token stands in its expert's list, nor on the batch.
-#include "common.cuh"
+#include "post_op.cuh"
 
 namespace lb {
 
@@ -94,8 +96,16 @@ __global__ void route_topk_kernel(int* __restrict__ ids, float* __restrict__ wei
 
 // ---- dispatch --------------------------------------------------------------------------------------------------
 // meta: [0] number of row tiles, then (expert, first place, end place) per tile from meta[4] on.
-__global__ void expert_dispatch_kernel(const int* __restrict__ ids, int pairs, int experts, int tile_rows, int* __restrict__ offsets,
-                                       int* __restrict__ pair_at, int* __restrict__ place_of, int* __restrict__ meta) {
+// tokens: null, or the step's token ids; ids is then the table [vocab, top] and pair i is choice i % top of token i / top.
+__device__ __forceinline__ int expert_of(const int* ids, const int* tokens, int top, int i) {
+  if (tokens == nullptr) return ids[i];
+  const int t = i / top;
+  return ids[(size_t)tokens[t] * top + (i - t * top)];
+}
+
+__global__ void expert_dispatch_kernel(const int* __restrict__ ids, const int* __restrict__ tokens, int top, int pairs, int experts,
+                                       int tile_rows, int* __restrict__ offsets, int* __restrict__ pair_at,
+                                       int* __restrict__ place_of, int* __restrict__ meta) {
   extern __shared__ int ism[];
   pdl_trigger();
   pdl_wait();
@@ -105,7 +115,7 @@ __global__ void expert_dispatch_kernel(const int* __restrict__ ids, int pairs, i
   for (int e = threadIdx.x; e < experts; e += blockDim.x) count[e] = 0;
   __syncthreads();
   // a pair's rank among its expert's pairs: whatever order the atomics give; the order never shows in a result
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) place_of[i] = atomicAdd(&count[ids[i]], 1);
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) place_of[i] = atomicAdd(&count[expert_of(ids, tokens, top, i)], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int a = 0, tl = 0;
@@ -119,7 +129,7 @@ __global__ void expert_dispatch_kernel(const int* __restrict__ ids, int pairs, i
   __syncthreads();
   for (int e = threadIdx.x; e <= experts; e += blockDim.x) offsets[e] = start[e];
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int place = start[ids[i]] + place_of[i];
+    const int place = start[expert_of(ids, tokens, top, i)] + place_of[i];
     place_of[i] = place;
     pair_at[place] = i;
   }
@@ -135,7 +145,8 @@ __global__ void expert_dispatch_kernel(const int* __restrict__ ids, int pairs, i
 // The same sort with every expert's run padded to whole tiles of `tile` places, for products that take their rows
 // from a matrix by whole tiles (the tensor-memory product): place_of [pairs], pair_at [places] (-1 where a place is
 // padding), tile_group [places / tile] (the expert of each tile; the tiles behind the last run name expert 0 and hold padding).
-__global__ void expert_dispatch_padded_kernel(const int* __restrict__ ids, int pairs, int experts, int tile, int places,
+__global__ void expert_dispatch_padded_kernel(const int* __restrict__ ids, const int* __restrict__ tokens, int top, int pairs,
+                                              int experts, int tile, int places,
                                               int* __restrict__ pair_at, int* __restrict__ place_of, int* __restrict__ tile_group) {
   extern __shared__ int ism[];
   pdl_trigger();
@@ -146,7 +157,7 @@ __global__ void expert_dispatch_padded_kernel(const int* __restrict__ ids, int p
   for (int i = threadIdx.x; i < places; i += blockDim.x) pair_at[i] = -1;
   for (int i = threadIdx.x; i < places / tile; i += blockDim.x) tile_group[i] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) place_of[i] = atomicAdd(&count[ids[i]], 1);
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) place_of[i] = atomicAdd(&count[expert_of(ids, tokens, top, i)], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int a = 0;
@@ -155,7 +166,7 @@ __global__ void expert_dispatch_padded_kernel(const int* __restrict__ ids, int p
   }
   __syncthreads();
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int place = start[ids[i]] + place_of[i];
+    const int place = start[expert_of(ids, tokens, top, i)] + place_of[i];
     place_of[i] = place;
     pair_at[place] = i;
   }
@@ -198,6 +209,7 @@ struct ExpertGemmParams {
   long long ldx, ldy;
   int gather;               // 1: x row of a place = pair_at[place] / top; 0: the place
   int gated, act; float limit;
+  int post;                 // not gated: an element operation (post_op.cuh) on the sums
   int interleaved;          // gated only: gate and up rows alternate in blocks of 64 (gate rows of 64 features, then their up rows)
 };
 
@@ -280,7 +292,7 @@ __global__ void __launch_bounds__(256) expert_gemm_plain_kernel(ExpertGemmParams
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tc * 4 + j;
       if (gn >= ncols) continue;
-      const float v = GATED ? expert_act(p.act, p.limit, acc[i][j], acc2[i][j]) : acc[i][j];
+      const float v = GATED ? expert_act(p.act, p.limit, acc[i][j], acc2[i][j]) : post_op(p.post, 0.f, acc[i][j]);
       y[(size_t)place * p.ldy + gn] = from_f32<TY>(v);
     }
   }
@@ -410,24 +422,35 @@ __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p
         for (int j = 0; j < 2; ++j) {
           const int n = n0 + wn + nb * 8 + 2 * t4 + j;
           if (n >= ncols) continue;
-          const float v = GATED ? expert_act(p.act, p.limit, acc[mi][nb][2 * half + j], acc2[mi][nb][2 * half + j]) : acc[mi][nb][2 * half + j];
+          const float v = GATED ? expert_act(p.act, p.limit, acc[mi][nb][2 * half + j], acc2[mi][nb][2 * half + j]) : post_op(p.post, 0.f, acc[mi][nb][2 * half + j]);
           y[(size_t)place * p.ldy + n] = from_f32<TY>(v);
         }
       }
 }
 
 // ---- combine ---------------------------------------------------------------------------------------------------
+// weights: null means `weight` for every pair.  gate (with x, the rows the products read): the always-used expert's output
+// counts times sigmoid(gate . x[t]).
 template <typename TO, typename TA>
-__global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restrict__ y, const float* __restrict__ weights,
-                                      const int* __restrict__ place_of, const TA* __restrict__ always, int top, int width) {
+__global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restrict__ y, const float* __restrict__ weights, float weight,
+                                      const int* __restrict__ place_of, const TA* __restrict__ always, const void* __restrict__ x,
+                                      int x_bf16, const float* __restrict__ gate, int top, int width) {
+  __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
+  float g = 1.f;
+  if (gate) {
+    float part = 0.f;
+    for (int j = threadIdx.x; j < width; j += blockDim.x)
+      part += (x_bf16 ? to_f32(((const bf16*)x)[(size_t)t * width + j]) : ((const float*)x)[(size_t)t * width + j]) * gate[j];
+    g = 1.f / (1.f + expf(-block_sum(part, scratch)));
+  }
   for (int j = threadIdx.x; j < width; j += blockDim.x) {
     float acc = 0.f;
     for (int k = 0; k < top; ++k)
-      acc = fmaf(weights[(size_t)t * top + k], y[(size_t)place_of[(size_t)t * top + k] * width + j], acc);
-    if (always) acc += to_f32(always[(size_t)t * width + j]);
+      acc = fmaf(weights ? weights[(size_t)t * top + k] : weight, y[(size_t)place_of[(size_t)t * top + k] * width + j], acc);
+    if (always) acc = fmaf(g, to_f32(always[(size_t)t * width + j]), acc);
     out[(size_t)t * width + j] = from_f32<TO>(acc);
   }
 }
@@ -454,24 +477,27 @@ LB_EXPORT int lb_route_topk(int* ids, float* weights, const float* logits, long 
 LB_EXPORT int lb_expert_tile_rows() { return lb::EX_BM; }
 
 // ids [pairs] -> offsets [experts + 1], pair_at [pairs], place_of [pairs], meta [4 + 3 * (pairs / tile_rows + experts)]
-LB_EXPORT int lb_expert_dispatch(const int* ids, int pairs, int experts, int* offsets, int* pair_at, int* place_of, int* meta,
-                                 cudaStream_t stream) {
+// (tokens != null: ids is the table [vocab, top] and pairs = tokens * top; its entries lie in 0 .. experts - 1)
+LB_EXPORT int lb_expert_dispatch(const int* ids, const int* tokens, int top, int pairs, int experts, int* offsets, int* pair_at,
+                                 int* place_of, int* meta, cudaStream_t stream) {
+  LB_CHECK_ARG(tokens == nullptr || (top > 0 && pairs % top == 0), "expert_dispatch: %d pairs are not %d choices a token", pairs, top);
   LB_CHECK_ARG(ids && offsets && pair_at && place_of && meta, "expert_dispatch: null argument");
   LB_CHECK_ARG(pairs >= 0 && experts > 0 && experts <= 4096, "expert_dispatch: bad sizes pairs=%d experts=%d", pairs, experts);
   static_assert(lb::EX_BM == lb::EM_BM, "both products walk the same row tiles");
   const size_t smem = (size_t)(3 * experts + 2) * sizeof(int);
-  lb::launch(lb::expert_dispatch_kernel, dim3(1), dim3(1024), smem, stream, ids, pairs, experts, (int)lb::EX_BM, offsets, pair_at, place_of, meta);
+  lb::launch(lb::expert_dispatch_kernel, dim3(1), dim3(1024), smem, stream, ids, tokens, top, pairs, experts, (int)lb::EX_BM, offsets, pair_at, place_of, meta);
   LB_CHECK_LAUNCH("expert_dispatch");
   return 0;
 }
 
 // places: a multiple of tile, at least pairs + experts * (tile - 1) rounded up to it
-LB_EXPORT int lb_expert_dispatch_padded(const int* ids, int pairs, int experts, int tile, int places, int* pair_at, int* place_of,
-                                        int* tile_group, cudaStream_t stream) {
+LB_EXPORT int lb_expert_dispatch_padded(const int* ids, const int* tokens, int top, int pairs, int experts, int tile, int places,
+                                        int* pair_at, int* place_of, int* tile_group, cudaStream_t stream) {
+  LB_CHECK_ARG(tokens == nullptr || (top > 0 && pairs % top == 0), "expert_dispatch_padded: %d pairs are not %d choices a token", pairs, top);
   LB_CHECK_ARG(ids && pair_at && place_of && tile_group, "expert_dispatch_padded: null argument");
   LB_CHECK_ARG(pairs >= 0 && experts > 0 && experts <= 4096 && tile > 0 && places % tile == 0 && places >= pairs + experts * (tile - 1),
                "expert_dispatch_padded: bad sizes pairs=%d experts=%d tile=%d places=%d", pairs, experts, tile, places);
-  lb::launch(lb::expert_dispatch_padded_kernel, dim3(1), dim3(1024), (size_t)(2 * experts + 1) * sizeof(int), stream, ids, pairs, experts,
+  lb::launch(lb::expert_dispatch_padded_kernel, dim3(1), dim3(1024), (size_t)(2 * experts + 1) * sizeof(int), stream, ids, tokens, top, pairs, experts,
              tile, places, pair_at, place_of, tile_group);
   LB_CHECK_LAUNCH("expert_dispatch_padded");
   return 0;
@@ -491,7 +517,8 @@ LB_EXPORT int lb_expert_gather_rows(void* xs, const void* x, const int* pair_at,
 // fast: 1 allows the tensor-core kernel (bfloat16 x and W, K a multiple of 8, 16-byte aligned rows).
 LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* meta,
                              const int* pair_at, int max_tiles, int N, int K, long long ldx, long long ldy, int top, int gather,
-                             int gated, int act, float limit, int fast, int interleaved, cudaStream_t stream) {
+                             int gated, int act, float limit, int fast, int interleaved, int post, cudaStream_t stream) {
+  LB_CHECK_ARG(lb::valid_post(post, 0.f) && !(post && gated), "expert_gemm: element operation %d", post);
   LB_CHECK_ARG(!interleaved || (gated && N % 128 == 0), "expert_gemm: interleaved gate and up rows come in blocks of 64");
   LB_CHECK_ARG(lb::valid_dtype(y_dtype) && lb::valid_dtype(x_dtype) && lb::valid_dtype(w_dtype), "expert_gemm: bad dtype");
   LB_CHECK_ARG(y && x && w && meta && pair_at && N > 0 && K > 0 && top > 0 && max_tiles >= 0 && (!gated || N % 2 == 0) && ldx >= K,
@@ -501,7 +528,7 @@ LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, c
   if (max_tiles == 0) return 0;
   lb::ExpertGemmParams p;
   p.y = y; p.x = x; p.w = w; p.meta = meta; p.pair_at = pair_at; p.N = N; p.K = K; p.top = top; p.ldx = ldx; p.ldy = ldy;
-  p.gather = gather; p.gated = gated; p.act = act; p.limit = limit; p.interleaved = interleaved;
+  p.gather = gather; p.gated = gated; p.act = act; p.limit = limit; p.interleaved = interleaved; p.post = post;
   const int ncols = gated ? N / 2 : N;
   const bool mma = fast && x_dtype == LB_BF16 && w_dtype == LB_BF16 && K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0;
   if (mma) {
@@ -513,11 +540,18 @@ LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, c
       cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<lb::bf16, false, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<false, 128>());
       cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<float, true, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<true, 64>());
       cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<lb::bf16, true, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<true, 64>());
+      cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<float, false, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<false, 64>());
+      cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<lb::bf16, false, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<false, 64>());
       attr_set = true;
     }
-    // few row tiles and a gated product (two weight rows a column): tiles of 64 columns, twice the CTAs for the same weights
-    const bool narrow = gated && (long long)max_tiles * ((ncols + 127) / 128) < 2 * 148;
-    if (narrow) {
+    // few row tiles: tiles of 64 columns, twice the CTAs for the same weights (a down product keeps the wide ones)
+    const bool narrow = (gated || post) && (long long)max_tiles * ((ncols + 127) / 128) < 2 * 148;
+    if (narrow && !gated) {
+      dim3 grid((ncols + 63) / 64, max_tiles);
+      LB_DISPATCH_DTYPE(y_dtype, TY, {
+        lb::launch(lb::expert_gemm_mma_kernel<TY, false, 64>, grid, dim3(256), lb::expert_mma_smem<false, 64>(), stream, p);
+      })
+    } else if (narrow) {
       dim3 grid((ncols + 63) / 64, max_tiles);
       LB_DISPATCH_DTYPE(y_dtype, TY, {
         lb::launch(lb::expert_gemm_mma_kernel<TY, true, 64>, grid, dim3(256), lb::expert_mma_smem<true, 64>(), stream, p);
@@ -544,16 +578,19 @@ LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, c
   return 0;
 }
 
-// out[t] = sum_k weights[t, k] * y[place_of[t, k]] (+ always[t]); y float32 [pairs, width]
-LB_EXPORT int lb_expert_combine(void* out, int out_dtype, const float* y, const float* weights, const int* place_of,
-                                const void* always, int always_dtype, int num_tokens, int top, int width, cudaStream_t stream) {
-  LB_CHECK_ARG(lb::valid_dtype(out_dtype) && lb::valid_dtype(always_dtype) && out && y && weights && place_of && top > 0 && width > 0, "expert_combine: bad arguments");
+// out[t] = sum_k weights[t, k] * y[place_of[t, k]] (+ always[t] [* sigmoid(gate . x[t])]); y float32 [pairs, width]; weights
+// null: every pair counts `weight`
+LB_EXPORT int lb_expert_combine(void* out, int out_dtype, const float* y, const float* weights, float weight, const int* place_of,
+                                const void* always, int always_dtype, const void* x, int x_dtype, const float* gate, int num_tokens,
+                                int top, int width, cudaStream_t stream) {
+  LB_CHECK_ARG(lb::valid_dtype(x_dtype) && (!gate || (x && always)), "expert_combine: a gate goes with the always-used expert and the sublayer's input");
+  LB_CHECK_ARG(lb::valid_dtype(out_dtype) && lb::valid_dtype(always_dtype) && out && y && place_of && top > 0 && width > 0, "expert_combine: bad arguments");
   if (num_tokens <= 0) return 0;
   const int threads = width >= 1024 ? 256 : 128;
   LB_DISPATCH_DTYPE(out_dtype, TO, {
     LB_DISPATCH_DTYPE(always_dtype, TA, {
-      lb::launch(lb::expert_combine_kernel<TO, TA>, dim3(num_tokens), dim3(threads), 0, stream, (TO*)out, y, weights, place_of,
-                 (const TA*)always, top, width);
+      lb::launch(lb::expert_combine_kernel<TO, TA>, dim3(num_tokens), dim3(threads), 0, stream, (TO*)out, y, weights, weight, place_of,
+                 (const TA*)always, x, x_dtype == LB_BF16 ? 1 : 0, gate, top, width);
     })
   })
   LB_CHECK_LAUNCH("expert_combine");

@@ -13,7 +13,9 @@
 // mixer whose heads each have a matrix of their own): batch b reads x + b * bx, w + b * bw and writes
 // y + b * by.  An optional gate (32-bit, [M, batches * N] with row stride ldg) multiplies element
 // (m, n) of batch b by sigmoid(gate[m, b * N + n]) before the single rounding.
-#include "common.cuh"
+//
+// lb_gemm_plain may apply one of the element operations of post_op.cuh to its 32-bit sums.
+#include "post_op.cuh"
 
 namespace lb {
 
@@ -23,7 +25,7 @@ template <typename TX, typename TW, typename TY>
 __global__ void __launch_bounds__(256)
 gemm_plain_kernel(TY* __restrict__ y, const TX* __restrict__ x, const TW* __restrict__ w, int M, int N,
                   int K, long long ldx, long long ldy, long long bx, long long bw, long long by,
-                  const float* __restrict__ gate, long long ldg) {
+                  const float* __restrict__ gate, long long ldg, int post, float post_c) {
   __shared__ float xs[PG_BK][PG_BM + 4];
   __shared__ float ws[PG_BK][PG_BN + 4];
   pdl_trigger();
@@ -73,6 +75,7 @@ gemm_plain_kernel(TY* __restrict__ y, const TX* __restrict__ x, const TW* __rest
       if (gn >= N) continue;
       float v = acc[i][j];
       if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)gm * ldg + gn]));
+      if (post) v = post_op(post, post_c, v);
       y[(size_t)gm * ldy + gn] = from_f32<TY>(v);
     }
   }
@@ -81,17 +84,18 @@ gemm_plain_kernel(TY* __restrict__ y, const TX* __restrict__ x, const TW* __rest
 template <typename TX, typename TW, typename TY>
 void launch_gemm_plain(void* y, const void* x, const void* w, int M, int N, int K, long long ldx,
                        long long ldy, cudaStream_t stream, int batches = 1, long long bx = 0, long long bw = 0,
-                       long long by = 0, const float* gate = nullptr, long long ldg = 0) {
+                       long long by = 0, const float* gate = nullptr, long long ldg = 0, int post = POST_NONE, float post_c = 0.f) {
   dim3 grid((N + PG_BN - 1) / PG_BN, (M + PG_BM - 1) / PG_BM, batches);
   launch(gemm_plain_kernel<TX, TW, TY>, grid, dim3(256), 0, stream, (TY*)y, (const TX*)x, (const TW*)w, M, N, K, ldx, ldy,
-         bx, bw, by, gate, ldg);
+         bx, bw, by, gate, ldg, post, post_c);
 }
 
 }  // namespace lb
 
 LB_EXPORT int lb_gemm_plain(void* y, int y_dtype, const void* x, int x_dtype, const void* w,
                             int w_dtype, int M, int N, int K, long long ldx, long long ldy,
-                            cudaStream_t stream) {
+                            int post, float post_c, cudaStream_t stream) {
+  LB_CHECK_ARG(lb::valid_post(post, post_c), "gemm_plain: unknown element operation %d (%f)", post, (double)post_c);
   LB_CHECK_ARG(lb::valid_dtype(y_dtype) && lb::valid_dtype(x_dtype) && lb::valid_dtype(w_dtype),
                "gemm_plain: bad dtype");
   LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && ldx >= K && ldy >= N, "gemm_plain: bad sizes M=%d N=%d K=%d", M, N, K);
@@ -100,7 +104,7 @@ LB_EXPORT int lb_gemm_plain(void* y, int y_dtype, const void* x, int x_dtype, co
   LB_DISPATCH_DTYPE(x_dtype, TX, {
     LB_DISPATCH_DTYPE(w_dtype, TW, {
       LB_DISPATCH_DTYPE(y_dtype, TY, {
-        lb::launch_gemm_plain<TX, TW, TY>(y, x, w, M, N, K, ldx, ldy, stream);
+        lb::launch_gemm_plain<TX, TW, TY>(y, x, w, M, N, K, ldx, ldy, stream, 1, 0, 0, 0, nullptr, 0, post, post_c);
       })
     })
   })

@@ -31,7 +31,7 @@
 // flag, stops, waits (bounded) for its loads in flight, frees its tensor memory and returns.
 // K must be a multiple of 8 and X, W 16-byte aligned (TMA strides); M, N, K tails are handled by
 // TMA's zero fill on loads and by bounds checks on stores.
-#include "common.cuh"
+#include "post_op.cuh"
 
 #include <cuda.h>
 #include <mutex>
@@ -269,6 +269,8 @@ struct GemmParams {
                         // features; the output has N/2 columns and holds act(gate) * up (computed in 32-bit) with
                         // act = silu (1), relu (2), the tanh form of gelu (3) or the clamped swish (4, see gated_mul)
   float act_limit = 0.f; // the clamp of activation 4
+  int post = POST_NONE;  // without swiglu: an element operation (post_op.cuh) on the 32-bit sums before they are stored
+  float post_c = 0.f;
   const int* tile_group = nullptr;   // many-token kernel only: w holds several matrices of N rows one below the other, and token
                                      // tile i (128 tokens) is multiplied with matrix tile_group[i] (tokens sorted into runs by
                                      // group, each run padded to whole tiles: the experts of a routed feed-forward)
@@ -476,7 +478,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
           for (int j = 0; j < 16; ++j) {
             const int m = m0 + c + j;
             if (m < p.M) {
-              const float v = (p.rs.on && direct) ? __uint_as_float(r[j]) * row_f[c + j] : __uint_as_float(r[j]);
+              float v = (p.rs.on && direct) ? __uint_as_float(r[j]) * row_f[c + j] : __uint_as_float(r[j]);
+              if (direct && p.post) v = post_op(p.post, p.post_c, v);
               if (!direct) part[(size_t)m * p.N + n] = v;
               else if (p.out_dtype == LB_F32) ((float*)p.y)[(size_t)m * p.ldy + n] = v;
               else ((bf16*)p.y)[(size_t)m * p.ldy + n] = __float2bfloat16_rn(v);
@@ -530,6 +533,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 float acc = 0.f;
 #pragma unroll
                 for (int z = 0; z < 16; ++z) acc += v[i][z];
+                if (p.post) acc = post_op(p.post, p.post_c, acc);
                 if (p.out_dtype == LB_F32) ((float*)p.y)[(size_t)(m + i) * p.ldy + n] = acc;
                 else ((bf16*)p.y)[(size_t)(m + i) * p.ldy + n] = __float2bfloat16_rn(acc);
               }
@@ -677,6 +681,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
           if (m >= p.M) break;
           float acc = cluster_sum_f32(base + (uint32_t)j * (BM * 4u), splits);
           if (p.rs.on) acc *= tok_rf[j - split * per];
+          if (p.post) acc = post_op(p.post, p.post_c, acc);
           if (p.out_dtype == LB_F32) ((float*)p.y)[(size_t)m * p.ldy + n] = acc;
           else ((bf16*)p.y)[(size_t)m * p.ldy + n] = __float2bfloat16_rn(acc);
         }
@@ -1125,6 +1130,13 @@ gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_x, const __g
 #pragma unroll
           for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * rf);
         }
+        if (p.post == POST_GELU) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(gelu_erf(__uint_as_float(r[j])));
+        } else if (p.post) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(post_op(p.post, p.post_c, __uint_as_float(r[j])));
+        }
         if (m < p.M && n < p.N) {
           if (vec_store && n + 16 <= p.N) {
             if (p.out_dtype == LB_F32) {
@@ -1309,7 +1321,7 @@ static int prefill_feature_tiles(const PrefillPlan& plan, int N) {
 static int launch_prefill(const void* y, int y_dtype, const void* x, const void* w, int M, int N, int K, long long ldx,
                           long long ldy, int swiglu, int force_bn, int pair, cudaStream_t stream,
                           const AddNormEpilogue* an = nullptr, const RowScale* rs = nullptr, float act_limit = 0.f,
-                          const int* tile_group = nullptr, int groups = 1) {
+                          const int* tile_group = nullptr, int groups = 1, int post = POST_NONE, float post_c = 0.f) {
   bool use_pair; int m_tiles, slots; PrefillPlan plan;
   if (tile_group) pair = 1;               // a group's run of tokens is padded to tiles of 128, not to pairs of them
   prefill_choose(M, N, K, swiglu, force_bn, pair, &use_pair, &m_tiles, &slots, &plan);
@@ -1324,6 +1336,7 @@ static int launch_prefill(const void* y, int y_dtype, const void* x, const void*
   GemmParams p;
   p.y = const_cast<void*>(y); p.workspace = nullptr; p.counters = nullptr; p.M = M; p.N = N; p.K = K; p.ldy = ldy;
   p.out_dtype = y_dtype; p.cluster = 0; p.swiglu = swiglu; p.act_limit = act_limit; p.tile_group = tile_group;
+  p.post = post; p.post_c = post_c;
   if (an) {
     p.an = *an; p.an.on = 1;
     if (p.an.tiles != prefill_feature_tiles(plan, N)) { set_error("gemm_tcgen05: %d columns of partial sums, the plan has %d feature tiles", p.an.tiles, prefill_feature_tiles(plan, N)); return 1; }
@@ -1389,7 +1402,8 @@ LB_EXPORT void lb_gemm_tcgen05_prefill_plan(int M, int N, int swiglu, int num_sm
 // kernel with one more term in the weights' coordinate; swiglu and act_limit as in lb_gemm_tcgen05.
 LB_EXPORT int lb_gemm_tcgen05_grouped(void* y, int y_dtype, const void* x, const void* w, int M, int N, int K, long long ldx,
                                       long long ldy, int swiglu, float act_limit, const int* tile_group, int groups,
-                                      cudaStream_t stream) {
+                                      int post, cudaStream_t stream) {
+  LB_CHECK_ARG(lb::valid_post(post, 0.f) && !(post && swiglu), "gemm_tcgen05_grouped: element operation %d", post);
   LB_CHECK_ARG(lb::valid_dtype(y_dtype) && tile_group && groups > 0, "gemm_tcgen05_grouped: bad arguments");
   LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && ldx >= K && ldy >= (swiglu ? N / 2 : N), "gemm_tcgen05_grouped: bad sizes M=%d N=%d K=%d", M, N, K);
   LB_CHECK_ARG(!swiglu || N % 128 == 0, "gemm_tcgen05_grouped: the fused activation needs gate and up rows in blocks of 64 (N=%d)", N);
@@ -1397,7 +1411,7 @@ LB_EXPORT int lb_gemm_tcgen05_grouped(void* y, int y_dtype, const void* x, const
                "gemm_tcgen05_grouped: K and the row stride must be multiples of 8, the operands 16-byte aligned");
   LB_CHECK_ARG((long long)N * groups < (1ll << 31), "gemm_tcgen05_grouped: too many weight rows");
   if (M == 0) return 0;
-  if (int rc = lb::launch_prefill(y, y_dtype, x, w, M, N, K, ldx, ldy, swiglu, 0, 1, stream, nullptr, nullptr, act_limit, tile_group, groups)) return rc;
+  if (int rc = lb::launch_prefill(y, y_dtype, x, w, M, N, K, ldx, ldy, swiglu, 0, 1, stream, nullptr, nullptr, act_limit, tile_group, groups, post)) return rc;
   LB_CHECK_LAUNCH("gemm_tcgen05_grouped");
   return 0;
 }
@@ -1438,12 +1452,14 @@ LB_EXPORT int lb_gemm_tcgen05_plan(int M, int N, int K, int* bt) {
 // row stride ldy.  workspace (float32, workspace_elems elements) and counters (int32, zero, counters_len
 // entries) are needed when K is split; with too little of either the product runs unsplit.
 // force_bt / force_splits (0: choose) are for tests.
+// post, post_c: an element operation (post_op.cuh) on the sums; not together with swiglu.
 // row_scale (may be null): the rows of x lack their norm's factor (see RowScale); taken by the few-token product with
 // the fused SwiGLU only.
 LB_EXPORT int lb_gemm_tcgen05(void* y, int y_dtype, const void* x, const void* w, int M, int N, int K, long long ldx,
                               long long ldy, float* workspace, long long workspace_elems, int* counters,
                               int counters_len, int force_bt, int force_splits, int swiglu, const lb::RowScale* row_scale,
-                              float act_limit, cudaStream_t stream) {
+                              float act_limit, int post, float post_c, cudaStream_t stream) {
+  LB_CHECK_ARG(lb::valid_post(post, post_c) && !(post && swiglu), "gemm_tcgen05: element operation %d (%f)", post, (double)post_c);
   LB_CHECK_ARG(!row_scale || (row_scale->sumsq && row_scale->tiles > 0), "gemm_tcgen05: a row scale without partial sums");
   LB_CHECK_ARG(lb::valid_dtype(y_dtype), "gemm_tcgen05: bad output dtype %d", y_dtype);
   LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && ldx >= K && ldy >= (swiglu ? N / 2 : N), "gemm_tcgen05: bad sizes M=%d N=%d K=%d", M, N, K);
@@ -1469,7 +1485,7 @@ LB_EXPORT int lb_gemm_tcgen05(void* y, int y_dtype, const void* x, const void* w
     LB_CHECK_ARG(force_splits == 0 || (fw >= 16 && fw <= lb::PF_BN && fw % 16 == 0 && (!swiglu || fw % 128 == 0)),
                  "gemm_tcgen05: tile width %d is no multiple of 16 (128 with SwiGLU) up to 256", fw);
     LB_CHECK_ARG(force_bt >= -2, "gemm_tcgen05: token tile %d is not one of 16, 32, 64, 128, 256", force_bt);
-    if (int rc = lb::launch_prefill(y, y_dtype, x, w, M, N, K, ldx, ldy, swiglu, force_splits, -force_bt, stream, nullptr, row_scale, act_limit)) return rc;
+    if (int rc = lb::launch_prefill(y, y_dtype, x, w, M, N, K, ldx, ldy, swiglu, force_splits, -force_bt, stream, nullptr, row_scale, act_limit, nullptr, 1, post, post_c)) return rc;
     LB_CHECK_LAUNCH("gemm_tcgen05 (many tokens)");
     return 0;
   }
@@ -1503,7 +1519,7 @@ LB_EXPORT int lb_gemm_tcgen05(void* y, int y_dtype, const void* x, const void* w
   // Clusters when the split count allows it and the caller did not ask for the workspace path
   // (force_splits < 0 asks for -force_splits splits through the workspace).
   p.cluster = (!workspace_path && splits > 1 && splits <= 8) ? splits : 0;
-  p.swiglu = swiglu; p.act_limit = act_limit;
+  p.swiglu = swiglu; p.act_limit = act_limit; p.post = post; p.post_c = post_c;
   LB_CHECK_ARG(!row_scale || splits == 1 || p.cluster > 0,
                "gemm_tcgen05: a row scale is not taken by a product that is split through the workspace (M=%d, %d splits)", M, splits);
   if (row_scale) { p.rs = *row_scale; p.rs.on = 1; }

@@ -521,7 +521,7 @@ class ModelRunner:
         step = StepContext(
             num_tokens=T, num_seqs=S, positions=d_pos, token_seq=d_seq, cu_tokens=d_cu, context_lens=d_ctx,
             block_tables=d_tables, state_slots=d_slots, q_lens=q_lens, start_positions=starts,
-            max_q_len=batch.max_q_len, max_context_len=max_ctx, span_hint=batch.span_hint, plans=plans)
+            max_q_len=batch.max_q_len, max_context_len=max_ctx, span_hint=batch.span_hint, plans=plans, token_ids=d_tok)
         self.rt.stream = self._stream()
         d_rows = d_rows if R else None
         d_fresh = d_fresh if has_state and (new_slots or shape is not None) else None

@@ -4,7 +4,8 @@
 called twice (with two caches), and a call may read a cache that an earlier call has written
 (`write_cache=False`): then the mixer computes queries only and attends to what is there.  A call may ask for the
 embedding's output to be added to the stream before its block runs (`add_embedding`: models that repeat a run of
-layers and feed the input in again at the start of every pass).
+layers and feed the input in again at the start of every pass), or name a pass that starts with it (`entry`: the model's
+stream entry then mixes the stream with the embedding's output, see parts/stream_entry.py).
 """
 from __future__ import annotations
 
@@ -14,8 +15,10 @@ from typing import Optional, Sequence
 import torch
 
 from .. import ops
-from ..parts.base import Block, KVPages, Norm, Part, Runtime, StateSlot, StepContext, StreamCopy
+from ..parts.base import Block, KVPages, Norm, Part, Pending, Runtime, StateSlot, StepContext, StreamCopy
 from ..parts.embedding import OutputHead, TokenEmbedding
+from ..parts.norm import pending_terms
+from ..parts.stream_entry import StreamEntry
 
 
 @dataclass(frozen=True)
@@ -24,6 +27,7 @@ class LayerCall:
     cache: int
     write_cache: bool = True
     add_embedding: bool = False      # the embedding's output is added to the stream before this call's block runs
+    entry: int = -1                  # >= 0: the number of the pass that starts here; the stream goes through the stream entry first
 
 
 class DecoderModel(Part):
@@ -31,8 +35,11 @@ class DecoderModel(Part):
 
     def __init__(self, rt: Runtime, embedding: TokenEmbedding, blocks: Sequence[Block], calls: Sequence[LayerCall],
                  final_norm: Norm, head: OutputHead, vocab_size: int, max_positions: int, eos_token_ids: Sequence[int] = (),
-                 ignored_names: Sequence[str] = ()):
+                 ignored_names: Sequence[str] = (), stream_entry: Optional[StreamEntry] = None):
         self.rt = rt
+        self.stream_entry = stream_entry
+        if any(c.entry >= 0 for c in calls) and (stream_entry is None or any(c.add_embedding for c in calls)):
+            raise ValueError("calls that start a pass need the model's stream entry, and feed the embedding in by it alone")
         self.embedding, self.blocks, self.calls = embedding, list(blocks), list(calls)
         self.final_norm, self.head = final_norm, head
         self.vocab_size, self.max_positions = vocab_size, max_positions
@@ -61,7 +68,7 @@ class DecoderModel(Part):
         self._writer = written
 
     def children(self) -> list[Part]:
-        return [self.embedding, *self.blocks, self.final_norm, self.head]
+        return [self.embedding, *([self.stream_entry] if self.stream_entry is not None else []), *self.blocks, self.final_norm, self.head]
 
     def ignored_names(self) -> list[str]:
         return self.head.ignored_names() + self._ignored
@@ -70,40 +77,52 @@ class DecoderModel(Part):
         """What each cache id has to hold, as asked by the block that writes it (its mixer's needs, and the block's own)."""
         return [self.blocks[self.calls[self._writer[j]].block].cache_request() for j in range(self.num_caches)]
 
+    def _settle(self, residual: torch.Tensor, delta) -> None:
+        """Add what a block left to the stream by a kernel of its own; nothing is left then."""
+        if isinstance(delta, Pending):
+            ops.stream_norm(residual, self.rt.stream, **pending_terms(delta))
+        elif torch.is_tensor(delta) or isinstance(delta, tuple):
+            for d in delta if isinstance(delta, tuple) else (delta,):
+                ops.add_into(residual, d, self.rt.stream)
+        elif delta is not None and not isinstance(delta, StreamCopy):
+            raise ops.KernelError("a block that hands its output on inside a product stands in front of one that cannot take it so")
+
     def forward(self, token_ids: torch.Tensor, step: StepContext, caches: Sequence[object],
                 logit_rows: Optional[torch.Tensor]) -> Optional[torch.Tensor]:
         """Run the tokens of one step; float32 logits [R, vocab] for the rows asked for (None if none)."""
+        step.memo.clear()
         again = None                                     # a second copy of the embedding's output, for the calls that add it
         if any(c.add_embedding for c in self.calls):
             again = self.rt.empty((token_ids.shape[0], self.embedding.hidden_size), torch.float32)
+        enters = any(c.entry >= 0 for c in self.calls)
+        if enters:
+            again = self.rt.empty((token_ids.shape[0], self.embedding.hidden_size))
         pos = step.positions if getattr(self.embedding, "uses_positions", False) else None
         residual = self.embedding.forward(token_ids, pos, copy=again) if again is not None else (
             self.embedding.forward(token_ids, pos) if pos is not None else self.embedding.forward(token_ids))
         delta = None
+        from_embedding = self.stream_entry.embedding_half(again) if enters else None
         for i, c in enumerate(self.calls):
+            if c.entry >= 0:
+                if not isinstance(delta, Pending):
+                    delta = self._settle(residual, delta)
+                residual, delta = self.stream_entry.forward(residual, delta, from_embedding, c.entry)
             if c.add_embedding:
                 # with what the block before left, if this block's first norm adds two things in its pass; else by itself
                 if self.blocks[c.block].takes_delta_parts and (delta is None or (torch.is_tensor(delta) and delta.dtype == again.dtype)):
                     delta = (delta, again) if delta is not None else (again,)
                 else:
-                    if isinstance(delta, tuple):
-                        for d in delta:
-                            ops.add_into(residual, d, self.rt.stream)
-                        delta = None
-                    elif torch.is_tensor(delta):
-                        ops.add_into(residual, delta, self.rt.stream)
-                        delta = None
-                    elif delta is not None and not isinstance(delta, StreamCopy):
-                        raise ops.KernelError("the embedding cannot be added again behind a block that hands its output on inside a product")
+                    delta = self._settle(residual, delta)
                     ops.add_into(residual, again, self.rt.stream)
-                    delta = None
             # what the call after this one offers to take over from this one's last product (see Block.entry_sink)
             nxt = self.calls[i + 1] if i + 1 < len(self.calls) else None
             block = self.blocks[c.block]
             if isinstance(delta, StreamCopy) and not block.takes_stream_copy:
                 delta = None                             # nothing is left to be added; this block makes its own input
+            if isinstance(delta, Pending) and not block.takes_pending:
+                delta = self._settle(residual, delta)
             next_sink = (self.blocks[nxt.block].entry_sink(residual, step.num_tokens, nxt.write_cache)
-                         if nxt is not None and not nxt.add_embedding else None)
+                         if nxt is not None and not nxt.add_embedding and nxt.entry < 0 else None)
             # a block whose sublayers run side by side may leave their outputs unsummed when the norm that adds them
             # to the residual stream takes both (see Block.offers_delta_parts)
             parts_ok = (self.blocks[nxt.block].takes_delta_parts if nxt is not None else self.final_norm.takes_delta_parts)
@@ -117,5 +136,7 @@ class DecoderModel(Part):
             return None
         if isinstance(delta, StreamCopy):
             delta = None
+        if isinstance(delta, Pending) and not self.final_norm.takes_pending:
+            delta = self._settle(residual, delta)
         h = self.final_norm.add_forward(residual, delta, self.rt.act_dtype, rows=logit_rows)
         return self.head.forward(h)

@@ -31,7 +31,10 @@ def dtype_code(dt: torch.dtype) -> int:
 
 _SIGNATURES = {
     "lb_embedding": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p,
-                     c_void_p],
+                     c_int, c_void_p],
+    "lb_stream_norm": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p,
+                       c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                       c_int, c_void_p],
     "lb_layernorm": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "lb_layernorm_add": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_float, c_float, c_void_p, c_int,
                          c_int, c_int, c_void_p],
@@ -42,14 +45,15 @@ _SIGNATURES = {
                          c_int, c_longlong, c_void_p],
     "lb_head_gate": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_longlong, c_float, c_int, c_int, c_int, c_void_p],
     "lb_route_topk": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
-    "lb_expert_dispatch": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+    "lb_expert_dispatch": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "lb_expert_gemm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong,
-                       c_longlong, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p],
-    "lb_expert_dispatch_padded": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+                       c_longlong, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+    "lb_expert_dispatch_padded": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "lb_expert_gather_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lb_gemm_tcgen05_grouped": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_float,
-                                c_void_p, c_int, c_void_p],
-    "lb_expert_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+                                c_void_p, c_int, c_int, c_void_p],
+    "lb_expert_combine": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int,
+                          c_int, c_int, c_void_p],
     "lb_add_group_rmsnorm": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
                              c_float, c_void_p],
     "lb_scale": [c_void_p, c_longlong, c_float, c_void_p],
@@ -67,7 +71,7 @@ _SIGNATURES = {
     "lb_add_rmsnorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "lb_rope_kv": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_void_p,
                    c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_void_p],
+                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int, c_void_p],
     "lb_rotate_rows": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int,
                        c_float, c_void_p],
     "lb_round_cols": [c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p],
@@ -92,9 +96,9 @@ _SIGNATURES = {
     "lb_activation": [c_int, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_float, c_float, c_void_p],
     "lb_swiglu": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_float, c_void_p],
     "lb_gemm_plain": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_longlong,
-                      c_longlong, c_void_p],
+                      c_longlong, c_int, c_float, c_void_p],
     "lb_gemm_tcgen05": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_void_p,
-                        c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
+                        c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_int, c_float, c_void_p],
     "lb_gemm_tcgen05_addnorm": [c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p,
                                 c_int, c_void_p],
     "lb_upload": [c_void_p, c_void_p, c_longlong, c_void_p],
@@ -104,9 +108,9 @@ _SIGNATURES = {
                            c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p, c_void_p],
     "lb_attention_flash_ex": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                               c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p,
-                              c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
+                              c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lb_attention_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_void_p],
+                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_float, c_void_p],
     "lb_sample": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
 }
 
@@ -164,9 +168,9 @@ def embedding(out: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, stream:
               sin_freq: torch.Tensor | None = None, scale: float = 1.0, copy: torch.Tensor | None = None) -> None:
     """out[t, :] = table[ids[t], :] * scale as float32; with a table of position vectors, + pos_table[positions[t], :]; with
     `sin_freq` (float64 [ceil(H / 2)]) instead + the sinusoidal vector whose entries 2i, 2i + 1 are the sine and
-    cosine of positions[t] * sin_freq[i].  `copy` (float32, out's shape) receives the same rows a second time."""
+    cosine of positions[t] * sin_freq[i].  `copy` (out's shape, either type) receives the same rows a second time."""
     if copy is not None:
-        _check(copy, "embedding copy", torch.float32)
+        _check(copy, "embedding copy")
         if copy.shape != out.shape:
             raise KernelError("the embedding's second copy has the first one's shape")
     _check(out, "embedding output", torch.float32); _check(ids, "token ids", torch.int32); _check(table, "embedding table")
@@ -181,7 +185,7 @@ def embedding(out: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, stream:
             raise KernelError(f"position vectors have {pos_table.shape[1]} values, the embedding {H}")
     _call("lb_embedding", out.data_ptr(), ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype), T, H,
           table.shape[0], _ptr(pos_table), _ptr(positions), pos_table.shape[0] if pos_table is not None else 0, _ptr(sin_freq),
-          float(scale), _ptr(copy), stream)
+          float(scale), _ptr(copy), dtype_code(copy.dtype) if copy is not None else F32, stream)
 
 
 def add_group_rmsnorm(out: torch.Tensor, residual: torch.Tensor, deltas: tuple, weight: torch.Tensor, groups: int,
@@ -302,18 +306,80 @@ def add_rmsnorm(out: torch.Tensor, residual: torch.Tensor, delta: torch.Tensor |
           dtype_code(delta.dtype) if delta is not None else F32, weight.data_ptr(), _ptr(rows), n, H, eps, stream)
 
 
+def stream_norm(residual: torch.Tensor, stream: int, out: torch.Tensor | None = None, weight: torch.Tensor | None = None, eps: float = 0.0,
+                parts: tuple | None = None, rows: torch.Tensor | None = None, adds: tuple = (), vec: torch.Tensor | None = None,
+                y: torch.Tensor | None = None, y_weight: torch.Tensor | None = None, y_eps: float = 0.0, experts=None) -> None:
+    """v = residual + adds + vec + y / sqrt(mean(y^2) + y_eps) * y_weight, row by row in 32-bit; residual = v (unless `rows` picks rows
+    or `parts` are asked for); then out = v / sqrt(mean(v^2) + eps) * weight, or parts = (hi, lo): v in two bfloat16 parts.
+    adds: up to two float32 matrices of the residual's shape; vec: one float32 row for all; y: a sublayer's output.  Instead
+    of y, `experts` = (rows [places, width] float32, place_of [T, top], weights [T, top] float32 or one number,
+    shared output or None, gate's input [T, width] or None, gate's weights [width] float32 or None): y = the weighted sum
+    of the token's experts' rows, plus the shared output times sigmoid(gate weights . gate's input)."""
+    _check(residual, "residual", torch.float32)
+    H = residual.shape[1]
+    for t in adds:
+        _check(t, "addend", torch.float32)
+        if t.shape != residual.shape:
+            raise KernelError("an addend has the residual's shape")
+    if len(adds) > 2:
+        raise KernelError("at most two addends")
+    for t, what in ((vec, "vector"), (y_weight, "norm weight"), (weight, "norm weight")):
+        if t is not None:
+            _check(t, what, torch.float32)
+            if t.numel() != H:
+                raise KernelError(f"a {what} of {t.numel()} for rows of {H}")
+    if rows is not None:
+        _check(rows, "row index", torch.int32)
+    lo = None
+    if parts is not None:
+        out, lo = parts
+        _check(lo, "low part", torch.bfloat16)
+    n = residual.shape[0] if rows is None else rows.shape[0]
+    for t in (out, lo):
+        if t is not None:
+            _check(t, "norm output")
+            if tuple(t.shape) != (n, H):
+                raise KernelError(f"an output of {tuple(t.shape)} for {n} rows of {H}")
+    y_dtype, x_dtype = F32, F32
+    e = place_of = weights = shared = x = gate = None
+    top, w1 = 0, 0.0
+    if y is not None:
+        _check(y, "sublayer output")
+        if y.shape != residual.shape:
+            raise KernelError("a sublayer's output has the residual's shape")
+        y_dtype = dtype_code(y.dtype)
+    elif experts is not None:
+        e, place_of, weights, shared, x, gate = experts
+        _check(e, "experts' rows", torch.float32); _check(place_of, "places", torch.int32)
+        top = place_of.numel() // residual.shape[0]
+        if not torch.is_tensor(weights):
+            weights, w1 = None, float(weights)
+        for t, dt in ((weights, torch.float32), (gate, torch.float32), (shared, None), (x, None)):
+            if t is not None:
+                _check(t, "operand of the experts' sum", dt)
+        y_dtype = dtype_code(shared.dtype) if shared is not None else F32
+        x_dtype = dtype_code(x.dtype) if x is not None else F32
+    _call("lb_stream_norm", _ptr(out), dtype_code(out.dtype) if out is not None else F32, _ptr(lo), residual.data_ptr(),
+          _ptr(adds[0]) if adds else None, _ptr(adds[1]) if len(adds) > 1 else None, _ptr(vec), _ptr(y), y_dtype, _ptr(y_weight), y_eps,
+          _ptr(weight), eps, _ptr(rows), _ptr(e), _ptr(place_of), _ptr(weights), top, w1, _ptr(shared), _ptr(x), x_dtype, _ptr(gate),
+          n, H, stream)
+
+
 def rope_kv(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_out: torch.Tensor,
             positions: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, eps: float, stream: int,
             q_norm_w: torch.Tensor | None = None, k_norm_w: torch.Tensor | None = None,
             inv_freq: torch.Tensor | None = None, rot_dim: int = 0,
             k_cache: torch.Tensor | None = None, v_cache: torch.Tensor | None = None,
             token_seq: torch.Tensor | None = None, block_table: torch.Tensor | None = None, page_size: int = 0,
-            k_out: torch.Tensor | None = None, v_out: torch.Tensor | None = None, v_dim: int = 0, rot_scale: float = 1.0) -> None:
+            k_out: torch.Tensor | None = None, v_out: torch.Tensor | None = None, v_dim: int = 0, rot_scale: float = 1.0,
+            pairs: bool = False, unit: bool = False) -> None:
     """Per-head norm of q and k, rotation, and the write of k and v into pages (or into k_out, v_out).
 
     q_in, k_in and v_in are 2-d views whose rows may be column ranges of one wider matrix; they may be float32 where
     the heads are stored in bfloat16 (a product with 32-bit output).  `v_dim`: the size of a value head if it is not
-    head_dim (the value pool then has rows of that size).  `rot_scale` multiplies the rotation's sines and cosines."""
+    head_dim (the value pool then has rows of that size).  `rot_scale` multiplies the rotation's sines and cosines.
+    `pairs`: neighbours (2i, 2i + 1) are rotated together, not (i, i + rot_dim/2).  `unit`: behind the rotation every q and
+    k head is divided by sqrt(mean(x^2) + eps) (no norm weights then)."""
     T = q_in.shape[0]
     dt = q_out.dtype
     for t, w in ((q_in, "q"), (k_in, "k"), (v_in, "v")):
@@ -328,7 +394,8 @@ def rope_kv(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_out: t
     _call("lb_rope_kv", dtype_code(dt), q_in.data_ptr(), k_in.data_ptr(), v_in.data_ptr(), q_in.stride(0),
           k_in.stride(0), v_in.stride(0), q_out.data_ptr(), _ptr(k_out), _ptr(v_out), _ptr(k_cache), _ptr(v_cache),
           positions.data_ptr(), _ptr(token_seq), _ptr(block_table), _ptr(q_norm_w), _ptr(k_norm_w), _ptr(inv_freq),
-          T, num_q_heads, num_kv_heads, head_dim, rot_dim, page_size, max_pages, eps, dtype_code(q_in.dtype), v_dim, float(rot_scale), stream)
+          T, num_q_heads, num_kv_heads, head_dim, rot_dim, page_size, max_pages, eps, dtype_code(q_in.dtype), v_dim, float(rot_scale),
+          1 if pairs else 0, 1 if unit else 0, stream)
 
 
 def rotate_rows(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor | None, head_dim: int, rot_dim: int, ranges,
@@ -564,8 +631,13 @@ def swiglu(out: torch.Tensor, gate: torch.Tensor, up: torch.Tensor, stream: int,
           GATE_ACTS[act], limit, stream)
 
 
-def gemm_plain(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int) -> None:
-    """y[M, N] = x[M, K] . w[N, K]^T on the 32-bit pipes; x and y may be row-strided views."""
+# What a product may do with its 32-bit sums before they are rounded and stored (csrc/post_op.cuh): "gelu" is the exact form,
+# x / 2 (1 + erf(x / sqrt 2)); "cap" is c * tanh(x / c) with c = post_c.
+POST_OPS = {None: 0, "gelu": 1, "cap": 2}
+
+
+def gemm_plain(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, post: str | None = None, post_c: float = 0.0) -> None:
+    """y[M, N] = post(x[M, K] . w[N, K]^T) on the 32-bit pipes (see POST_OPS); x and y may be row-strided views."""
     M, K = x.shape
     N = w.shape[0]
     if w.shape[1] != K or tuple(y.shape) != (M, N):
@@ -573,7 +645,7 @@ def gemm_plain(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int) -
     if x.stride(1) != 1 or y.stride(1) != 1 or not w.is_contiguous() or not (x.is_cuda and w.is_cuda and y.is_cuda):
         raise KernelError("gemm operands must be on the GPU with unit column stride; w contiguous")
     _call("lb_gemm_plain", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), dtype_code(x.dtype), w.data_ptr(),
-          dtype_code(w.dtype), M, N, K, x.stride(0) if M > 1 else K, y.stride(0) if M > 1 else N, stream)
+          dtype_code(w.dtype), M, N, K, x.stride(0) if M > 1 else K, y.stride(0) if M > 1 else N, POST_OPS[post], float(post_c), stream)
 
 
 def sample(tokens: torch.Tensor, logits: torch.Tensor, stream: int, temperature: torch.Tensor | None = None,
@@ -626,14 +698,15 @@ def _row_scale(sumsq: torch.Tensor | None, width: int, eps: float):
 
 def gemm_tcgen05(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, force_bt: int = 0,
                  force_splits: int = 0, swiglu: bool = False, sumsq: torch.Tensor | None = None, eps: float = 0.0,
-                 act: str = "silu", limit: float = 0.0) -> None:
+                 act: str = "silu", limit: float = 0.0, post: str | None = None, post_c: float = 0.0) -> None:
     """y[M, N] = x[M, K] . w[N, K]^T on the tensor cores (tcgen05, accumulators in tensor memory).
 
     With `swiglu` the rows of w alternate in blocks of 64 between gate rows and up rows of the same 64
     features (see interleave_gate_up), and y[M, N/2] = act(x . gate^T) * (x . up^T), formed in the epilogue
     (act: one of GATE_ACTS; `limit` is the clamp of "clamped_swish").
     With `sumsq` [M, tiles] the rows of x lack the factor of an RMSNorm over K values: row m of the product is
-    multiplied by rsqrt(sum(sumsq[m]) / K + eps), before the activation if there is one (see gemm_tcgen05_addnorm)."""
+    multiplied by rsqrt(sum(sumsq[m]) / K + eps), before the activation if there is one (see gemm_tcgen05_addnorm).
+    `post`, `post_c` (without swiglu): an element operation in the epilogue, see POST_OPS."""
     M, K = x.shape
     N = w.shape[0]
     if w.shape[1] != K or tuple(y.shape) != (M, N // 2 if swiglu else N):
@@ -643,7 +716,8 @@ def gemm_tcgen05(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int,
     ws, counters = _gemm_scratch(x.device)
     _call("lb_gemm_tcgen05", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), w.data_ptr(), M, N, K,
           x.stride(0) if M > 1 else K, y.stride(0) if M > 1 else y.shape[1], ws.data_ptr(), ws.numel(), counters.data_ptr(),
-          counters.numel(), force_bt, force_splits, (1 + GATE_ACTS[act]) if swiglu else 0, _row_scale(sumsq, K, eps), limit, stream)
+          counters.numel(), force_bt, force_splits, (1 + GATE_ACTS[act]) if swiglu else 0, _row_scale(sumsq, K, eps), limit,
+          POST_OPS[post], float(post_c), stream)
 
 
 class LbHeadEpilogue(ctypes.Structure):
@@ -859,26 +933,34 @@ def expert_max_tiles(pairs: int, experts: int) -> int:
     return -(-pairs // expert_tile_rows()) + experts
 
 
+def _dispatch_pairs(ids: torch.Tensor, tokens: torch.Tensor | None) -> tuple[int, int]:
+    if tokens is None:
+        return ids.numel(), ids.shape[-1]
+    _check(tokens, "token ids", torch.int32)
+    return tokens.numel() * ids.shape[1], ids.shape[1]
+
+
 def expert_dispatch(ids: torch.Tensor, experts: int, offsets: torch.Tensor, pair_at: torch.Tensor, place_of: torch.Tensor,
-                    meta: torch.Tensor, stream: int) -> None:
+                    meta: torch.Tensor, stream: int, tokens: torch.Tensor | None = None) -> None:
     """Sort the (token, choice) pairs by expert, on the device: offsets [experts + 1], pair_at [pairs] (the pair at each
-    place), place_of [pairs], meta [4 + 3 * expert_max_tiles] (the row tiles of the products)."""
+    place), place_of [pairs], meta [4 + 3 * expert_max_tiles] (the row tiles of the products).  ids: the experts of the pairs, [T, top], or, with the step's
+    `tokens` [T], a table [vocab, top] whose row of a token's id holds the token's experts (entries in 0 .. experts - 1)."""
     for t, what in ((ids, "expert ids"), (offsets, "offsets"), (pair_at, "pair list"), (place_of, "places"), (meta, "tile list")):
         _check(t, what, torch.int32)
-    pairs = ids.numel()
+    pairs, top = _dispatch_pairs(ids, tokens)
     if offsets.numel() < experts + 1 or pair_at.numel() < pairs or place_of.numel() < pairs or meta.numel() < 4 + 3 * expert_max_tiles(pairs, experts):
         raise KernelError("expert_dispatch: an output is too small")
-    _call("lb_expert_dispatch", ids.data_ptr(), pairs, experts, offsets.data_ptr(), pair_at.data_ptr(), place_of.data_ptr(),
+    _call("lb_expert_dispatch", ids.data_ptr(), _ptr(tokens), top, pairs, experts, offsets.data_ptr(), pair_at.data_ptr(), place_of.data_ptr(),
           meta.data_ptr(), stream)
 
 
 def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, pair_at: torch.Tensor, top: int,
                 gather: bool, stream: int, act: str | None = None, limit: float = 0.0, fast: bool = True,
-                interleaved: bool = False) -> None:
+                interleaved: bool = False, post: str | None = None) -> None:
     """y[place] = x[row(place)] . w[e]^T for the places of every expert e (see expert_dispatch); w [experts, N, K].
     `gather`: row(place) is the pair's token, else the place.  With `act`, w[e] is N/2 gate rows then N/2 up rows (or,
     `interleaved`, blocks of 64 gate rows and their 64 up rows in turn, see interleave_gate_up) and y[place] =
-    act(gate) * up with N/2 columns."""
+    act(gate) * up with N/2 columns.  `post` (without act): an element operation on the sums, see POST_OPS."""
     _check(y, "expert output"); _check(x, "expert input"); _check(w, "expert weights")
     E, N, K = w.shape
     pairs = pair_at.numel()
@@ -887,7 +969,8 @@ def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.T
         raise KernelError(f"expert_gemm shapes do not fit: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     _call("lb_expert_gemm", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), dtype_code(x.dtype), w.data_ptr(), dtype_code(w.dtype),
           meta.data_ptr(), pair_at.data_ptr(), expert_max_tiles(pairs, E), N, K, K, cols, top, 1 if gather else 0,
-          1 if act is not None else 0, GATE_ACTS[act] if act is not None else 0, limit, 1 if fast else 0, 1 if interleaved else 0, stream)
+          1 if act is not None else 0, GATE_ACTS[act] if act is not None else 0, limit, 1 if fast else 0, 1 if interleaved else 0,
+          POST_OPS[post], stream)
 
 
 GROUP_TILE = 128          # token tile of the grouped tensor-memory product
@@ -899,15 +982,16 @@ def expert_padded_places(pairs: int, experts: int) -> int:
 
 
 def expert_dispatch_padded(ids: torch.Tensor, experts: int, pair_at: torch.Tensor, place_of: torch.Tensor, tile_group: torch.Tensor,
-                           stream: int) -> None:
+                           stream: int, tokens: torch.Tensor | None = None) -> None:
     """Sort the pairs by expert with every run padded to whole tiles: pair_at [places] (-1: padding), place_of [pairs],
-    tile_group [places / GROUP_TILE] (the expert of each tile), places = expert_padded_places(pairs, experts)."""
+    tile_group [places / GROUP_TILE] (the expert of each tile), places = expert_padded_places(pairs, experts).
+    `tokens`: as in expert_dispatch."""
     for t, what in ((ids, "expert ids"), (pair_at, "pair list"), (place_of, "places"), (tile_group, "tile list")):
         _check(t, what, torch.int32)
-    pairs, places = ids.numel(), pair_at.numel()
+    (pairs, top), places = _dispatch_pairs(ids, tokens), pair_at.numel()
     if places != expert_padded_places(pairs, experts) or place_of.numel() < pairs or tile_group.numel() < places // GROUP_TILE:
         raise KernelError("expert_dispatch_padded: an output has the wrong size")
-    _call("lb_expert_dispatch_padded", ids.data_ptr(), pairs, experts, GROUP_TILE, places, pair_at.data_ptr(), place_of.data_ptr(),
+    _call("lb_expert_dispatch_padded", ids.data_ptr(), _ptr(tokens), top, pairs, experts, GROUP_TILE, places, pair_at.data_ptr(), place_of.data_ptr(),
           tile_group.data_ptr(), stream)
 
 
@@ -920,9 +1004,10 @@ def expert_gather_rows(xs: torch.Tensor, x: torch.Tensor, pair_at: torch.Tensor,
 
 
 def gemm_tcgen05_grouped(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, stream: int,
-                         act: str | None = None, limit: float = 0.0) -> None:
+                         act: str | None = None, limit: float = 0.0, post: str | None = None) -> None:
     """y[m] = x[m] . w[g]^T with g = tile_group[m // GROUP_TILE], on the tensor cores (the many-token kernel of gemm_tcgen05);
-    w [groups, N, K] bfloat16.  With `act`, w[g] holds gate and up rows interleaved in blocks of 64 and y = act(gate) * up."""
+    w [groups, N, K] bfloat16.  With `act`, w[g] holds gate and up rows interleaved in blocks of 64 and y = act(gate) * up.
+    `post` (without act): an element operation on the sums, see POST_OPS."""
     _check(y, "y"); _check(x, "x", torch.bfloat16); _check(w, "grouped weights", torch.bfloat16); _check(tile_group, "tile list", torch.int32)
     G, N, K = w.shape
     M = x.shape[0]
@@ -930,19 +1015,30 @@ def gemm_tcgen05_grouped(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, tile
     if x.shape[1] != K or tuple(y.shape) != (M, cols) or tile_group.numel() * GROUP_TILE < M:
         raise KernelError(f"gemm_tcgen05_grouped shapes do not fit: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     _call("lb_gemm_tcgen05_grouped", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), w.data_ptr(), M, N, K, K, cols,
-          (1 + GATE_ACTS[act]) if act is not None else 0, limit, tile_group.data_ptr(), G, stream)
+          (1 + GATE_ACTS[act]) if act is not None else 0, limit, tile_group.data_ptr(), G, POST_OPS[post], stream)
 
 
-def expert_combine(out: torch.Tensor, y: torch.Tensor, weights: torch.Tensor, place_of: torch.Tensor, stream: int,
-                   always: torch.Tensor | None = None) -> None:
-    """out[t] = sum_k weights[t, k] * y[place_of[t, k]] (+ always[t]), in 32-bit, k in order."""
-    _check(out, "combined output"); _check(y, "expert outputs", torch.float32); _check(weights, "expert weights", torch.float32)
-    _check(place_of, "places", torch.int32)
+def expert_combine(out: torch.Tensor, y: torch.Tensor, weights: torch.Tensor | float, place_of: torch.Tensor, stream: int,
+                   always: torch.Tensor | None = None, gate_input: torch.Tensor | None = None,
+                   gate_weight: torch.Tensor | None = None) -> None:
+    """out[t] = sum_k weights[t, k] * y[place_of[t, k]] (+ always[t], times sigmoid(gate_weight . gate_input[t]) if given), in
+    32-bit, k in order.  weights: [T, top], or one number for every pair."""
+    _check(out, "combined output"); _check(y, "expert outputs", torch.float32); _check(place_of, "places", torch.int32)
+    w1 = 0.0
+    if torch.is_tensor(weights):
+        _check(weights, "expert weights", torch.float32)
+    else:
+        weights, w1 = None, float(weights)
     if always is not None:
         _check(always, "shared expert output")
+    if gate_weight is not None:
+        _check(gate_weight, "gate weights", torch.float32); _check(gate_input, "gate input")
     T, W = out.shape
-    _call("lb_expert_combine", out.data_ptr(), dtype_code(out.dtype), y.data_ptr(), weights.data_ptr(), place_of.data_ptr(),
-          _ptr(always), dtype_code(always.dtype) if always is not None else F32, T, weights.shape[1], W, stream)
+    if T == 0:
+        return
+    _call("lb_expert_combine", out.data_ptr(), dtype_code(out.dtype), y.data_ptr(), _ptr(weights), w1, place_of.data_ptr(),
+          _ptr(always), dtype_code(always.dtype) if always is not None else F32, _ptr(gate_input),
+          dtype_code(gate_input.dtype) if gate_input is not None else F32, _ptr(gate_weight), T, place_of.numel() // T, W, stream)
 
 
 def zero_rows(state: torch.Tensor, slots: torch.Tensor, stream: int) -> None:
@@ -974,13 +1070,13 @@ def device_error() -> int:
             or int(lib.lb_attention_flash_device_error()))
 
 
-def linear(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, fast: bool) -> None:
-    """y = x . w^T.  `fast` allows the tensor-core kernel where its conditions hold (otherwise, and
+def linear(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, fast: bool, post: str | None = None, post_c: float = 0.0) -> None:
+    """y = post(x . w^T), see POST_OPS.  `fast` allows the tensor-core kernel where its conditions hold (otherwise, and
     always on the 32-bit path, the product runs on the ordinary pipes)."""
     if fast and gemm_tcgen05_ok(y, x, w):
-        gemm_tcgen05(y, x, w, stream)
+        gemm_tcgen05(y, x, w, stream, post=post, post_c=post_c)
     else:
-        gemm_plain(y, x, w, stream)
+        gemm_plain(y, x, w, stream, post=post, post_c=post_c)
 
 
 _attn_ws: dict[int, torch.Tensor] = {}
@@ -1006,9 +1102,10 @@ def _attention_workspace(device: torch.device, elems: int) -> torch.Tensor:
     return ws
 
 
-def attention_flash_ok(q: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int) -> bool:
-    """The conditions of the tensor-core attention kernel."""
-    return (q.dtype == torch.bfloat16 and head_dim % 8 == 0 and 8 <= head_dim <= 128
+def attention_flash_ok(q: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, v_dim: int = 0) -> bool:
+    """The conditions of the tensor-core attention kernels."""
+    v_dim = v_dim or head_dim
+    return (v_dim % 8 == 0 and 8 <= v_dim <= 128 and q.dtype == torch.bfloat16 and head_dim % 8 == 0 and 8 <= head_dim <= 128
             and num_q_heads % num_kv_heads == 0 and num_q_heads // num_kv_heads <= 64)
 
 
@@ -1067,7 +1164,7 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
                     splits: int, stream: int, force_workspace: bool = False, tma: bool = True, kv_share: int = 1,
                     slopes: torch.Tensor | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None, pool: int = 0,
                     pool_k: torch.Tensor | None = None, pool_v: torch.Tensor | None = None,
-                    pool_table: torch.Tensor | None = None, chunk: int = 0) -> None:
+                    pool_table: torch.Tensor | None = None, chunk: int = 0, v_dim: int = 0) -> None:
     """Tensor-core attention over pages.  tiles: int32 [n, 4] of (first token, tokens, request index, 0).
     `kv_share` > 1: the pools hold num_kv_heads / kv_share heads, and kv head j of this call reads pool head j // kv_share
     (many query heads on one cached head, cut into groups of at most 16 so that decoded tokens fit the decode kernel's tiles).
@@ -1075,9 +1172,9 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     kernel even where a cluster could combine them.  Tiles of at most 16 query rows (decoded tokens) over pages of
     8 to 128 tokens run in the kernel whose keys and values a warp of its own fetches by TMA; `tma=False` keeps them
     in the kernel that fetches with 16-byte copies, which takes every page size.  `softcap`, `sinks` and `pool` (with
-    pool_k, pool_v, pool_table) and `chunk` as in attention_plain; a launch with any of them runs in the kernel with
-    16-byte copies."""
-    if softcap > 0 or sinks is not None or pool or chunk:
+    pool_k, pool_v, pool_table) and `chunk` as in attention_plain; a launch with sinks, pooled blocks or chunks runs in the kernel
+    with 16-byte copies.  `v_dim`: the size of a value head if it is not head_dim (out is then [T, heads, v_dim])."""
+    if sinks is not None or pool or chunk:
         tma = False
     if sinks is not None:
         _check(sinks, "sinks", torch.float32)
@@ -1093,7 +1190,7 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
     by_tma = tma and max_rows <= 16 and page_size in (8, 16, 32, 64, 128)
     in_cluster = max_rows <= 16 and not force_workspace and (2 <= splits <= 8 or (splits <= 16 and by_tma))
     if splits > 1 and not in_cluster:
-        ws_elems = n * num_kv_heads * splits * max_rows * (head_dim + 2)
+        ws_elems = n * num_kv_heads * splits * max_rows * ((v_dim or head_dim) + 2)
         ws = _attention_workspace(q.device, ws_elems)
         ws_elems = ws.numel()
     _call("lb_attention_flash_ex", q.data_ptr(), out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
@@ -1101,7 +1198,7 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
           page_size, block_table.shape[1], k_cache.shape[0] if tma else 0, window, scale,
           -splits if force_workspace else splits, max_rows, _ptr(ws), ws_elems, kv_share, _ptr(slopes), softcap, _ptr(sinks),
           pool, _ptr(pool_k) if pool else None, _ptr(pool_v) if pool else None, _ptr(pool_table) if pool else None,
-          pool_table.shape[1] if pool else 0, int(chunk), stream)
+          pool_table.shape[1] if pool else 0, int(chunk), int(v_dim), stream)
 
 
 def attention_tcgen05_ok(q: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, page_size: int,
@@ -1138,7 +1235,7 @@ def attention_tcgen05_splits(num_tiles: int, num_kv_heads: int, max_span: int, s
 def attention_tcgen05(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       positions: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor, num_q_heads: int,
                       num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float, stream: int,
-                      key_splits: int = 1, slopes: torch.Tensor | None = None) -> None:
+                      key_splits: int = 1, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
     """Attention of portions of prompts on tcgen05 (S and O in tensor memory).  tiles: int32 [n, 4] of
     (first token, tokens, request index, 0) with tokens <= 2 * (128 // (nq // nkv)).  With key_splits > 1 the keys of
     every tile are cut into that many ranges, a CTA each, combined by a second kernel."""
@@ -1153,7 +1250,7 @@ def attention_tcgen05(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     _call("lb_attention_tcgen05", q.data_ptr(), out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
           positions.data_ptr(), block_table.data_ptr(), tiles.data_ptr(), tiles.shape[0], q.shape[0], num_q_heads,
           num_kv_heads, head_dim, page_size, k_cache.shape[0], block_table.shape[1], window, scale, key_splits,
-          _ptr(ws), ws_elems, _ptr(slopes), stream)
+          _ptr(ws), ws_elems, _ptr(slopes), float(softcap), stream)
 
 
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step, group: int,
@@ -1166,15 +1263,16 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     portions of prompts go to the tcgen05 kernel, the rest (decoded tokens, short portions, other head
     sizes) to the mma.sync kernels; everything else, and every step without a plan, goes to the plain kernel.
     `kv_share` > 1: the plan's lists other than "big" were made for groups of num_q_heads / (num_kv_heads * kv_share)
-    query heads, kv_share of which read one cached head (see attention_flash).  A capped score (`softcap`), sinks and
+    query heads, kv_share of which read one cached head (see attention_flash).  A capped score (`softcap`) is taken by
+    all of them, values of another size than the keys by all but the tcgen05 kernel.  Sinks and
     pooled blocks behind the window (`pool` tokens a block, their means in pool_k / pool_v, pages of group `pool_group`)
     and chunks (`chunk` = C: a query sees the keys of its own run of C positions only) run in the mma.sync kernel with
     16-byte copies, for portions and for decoded tokens, or in the plain kernel."""
-    extras = softcap > 0 or sinks is not None or pool > 0 or chunk > 0
+    extras = sinks is not None or pool > 0 or chunk > 0
+    v_dim = 0 if v_dim == head_dim else v_dim
     pool_table = step.block_tables[pool_group] if pool else None
-    if (plan is None or (v_dim and v_dim != head_dim) or ((slopes is not None or extras) and not scale > 0)
-            or (pool and kv_share != 1) or not attention_flash_ok(q, num_q_heads, num_kv_heads * kv_share, head_dim)):
-        # value heads of another size than the keys' are the plain kernel's alone
+    if (plan is None or ((slopes is not None or extras or softcap > 0) and not scale > 0)
+            or (pool and kv_share != 1) or not attention_flash_ok(q, num_q_heads, num_kv_heads * kv_share, head_dim, v_dim)):
         attention_plain(q, out, k_cache, v_cache, step.positions, step.token_seq, step.block_tables[group],
                         num_q_heads, num_kv_heads, head_dim, page_size, window, scale, stream, v_dim=v_dim, slopes=slopes,
                         softcap=softcap, sinks=sinks, pool=pool, pool_k=pool_k, pool_v=pool_v, pool_table=pool_table, chunk=chunk)
@@ -1189,18 +1287,18 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     kinds = ["all"]
     if slopes is not None:
         _check(slopes, "distance slopes", torch.float32)
-    if not extras and "big" in meta and attention_tcgen05_ok(q, num_q_heads, num_kv_heads, head_dim, page_size,
+    if not extras and not v_dim and "big" in meta and attention_tcgen05_ok(q, num_q_heads, num_kv_heads, head_dim, page_size,
                                                              step.block_tables[group].shape[1]):
         attention_tcgen05(q, out, k_cache, v_cache, step.positions, step.block_tables[group], meta["big"],
                           num_q_heads, num_kv_heads, head_dim, page_size, window, scale, stream,
-                          key_splits=attention_tcgen05_splits(meta["big"].shape[0], num_kv_heads, span), slopes=slopes)
+                          key_splits=attention_tcgen05_splits(meta["big"].shape[0], num_kv_heads, span), slopes=slopes, softcap=softcap)
         kinds = ["rest"] if "rest" in meta else []
     for kind in kinds:
         tiles = meta[kind]
         rows = min(most_rows[kind], 64)
-        wide = attention_wide_clusters(head_dim) if rows <= 16 and page_size in (8, 16, 32, 64, 128) and not extras else 0
+        wide = attention_wide_clusters(max(head_dim, v_dim)) if rows <= 16 and page_size in (8, 16, 32, 64, 128) and not extras else 0
         splits = attention_splits(tiles.shape[0], num_kv_heads * kv_share, span, rows, wide_clusters=wide)
         attention_flash(q, out, k_cache, v_cache, step.positions, step.block_tables[group], tiles, rows,
                         num_q_heads, num_kv_heads * kv_share, head_dim, page_size, window, scale, splits, stream, kv_share=kv_share,
                         slopes=slopes, softcap=softcap, sinks=sinks, pool=pool, pool_k=pool_k, pool_v=pool_v, pool_table=pool_table,
-                        chunk=chunk)
+                        chunk=chunk, v_dim=v_dim)

@@ -1,10 +1,10 @@
 from .base import (BatchShape, Block, FeedForward, KVCacheView, KVPages, Mixer, Norm, NormSink, ParamSpec, Part, PlanView,
                    PositionEncoding, RowScaled, Runtime, StateCacheView, StateSlot, StepContext, StepPlan)
-from .attention import GatedBiasAttention, GQAttention, distance_slopes
-from .block import ParallelBlock, PostNormBlock, PreNormBlock
+from .attention import CappedWindowAttention, GatedBiasAttention, GQAttention, distance_slopes
+from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
 from .causal_taps import CausalTaps
 from .decay_attention import DecayLinearAttention
-from .experts import RoutedExperts
+from .experts import RoutedExperts, TableExperts
 from .side_by_side import SideBySideMixer
 from .gated_recurrence import GatedLinearRecurrence
 from .latent_attention import LatentAttention
@@ -12,7 +12,8 @@ from .embedding import OutputHead, TokenEmbedding
 from .linear import Linear
 from .mlp import GatedFeedForward, SwiGLUFeedForward
 from .norm import GroupRMSNorm, LayerNorm, RMSNorm
-from .rope import RotaryEmbedding
+from .rope import NeighbourRotary, RotaryEmbedding
+from .stream_entry import StreamEntry
 
 __all__ = [
     "BatchShape", "Block", "FeedForward", "KVCacheView", "KVPages", "Mixer", "Norm", "NormSink", "ParamSpec", "Part", "PlanView",
@@ -20,4 +21,5 @@ __all__ = [
     "TokenEmbedding", "Linear", "SwiGLUFeedForward", "RMSNorm", "RotaryEmbedding", "ParallelBlock", "CausalTaps",
     "GatedLinearRecurrence", "LatentAttention", "GatedFeedForward", "GroupRMSNorm", "GatedBiasAttention", "distance_slopes",
     "PostNormBlock", "DecayLinearAttention", "RoutedExperts", "SideBySideMixer", "LayerNorm",
+    "CappedWindowAttention", "SandwichNormBlock", "TableExperts", "NeighbourRotary", "StreamEntry",
 ]

@@ -22,6 +22,7 @@ from .. import ops
 from .base import (BatchShape, KVCacheView, KVPages, Mixer, NormSink, ParamSpec, Part, PositionEncoding, RowScaled, Runtime,
                    StepContext, StepPlan)
 from .linear import Linear
+from .rope import NeighbourRotary
 
 # Entries with at least this many tokens in a step go to the tensor-memory attention kernel (128-row tiles).
 BIG_PORTION = 16
@@ -395,7 +396,7 @@ class PooledWindowAttention(Mixer):
 def _attention_plan_key(rt: Runtime, heads: int, kv_heads: int, dim: int, vdim: int) -> Optional[Hashable]:
     """The tile lists of the tensor-core kernels, as GQAttention's: they depend on the group size alone."""
     g = heads // kv_heads
-    return ("attention tiles", g) if rt.fast_kernels and g <= TILE_ROWS and vdim == dim else None
+    return ("attention tiles", g) if rt.fast_kernels and g <= TILE_ROWS and max(dim, vdim) <= 128 and dim % 8 == vdim % 8 == 0 else None
 
 
 def _attention_plan(batch: BatchShape, heads: int, kv_heads: int) -> StepPlan:
@@ -572,6 +573,76 @@ class GatedWindowAttention(Mixer):
                       plan=step.plans.get(self.plan_key()), v_dim=V if V != D else 0)
         # an elementwise gate is a gate of one number a "head" of one entry
         ops.head_gate(out, heads.view(T, H * V, 1), pre[:, c3:c3 + H * V], out_scale, rt.stream)
+
+    def forward(self, h: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
+        pre = self.proj.forward(h, out_dtype=torch.float32)
+        inner = self.rt.empty((h.shape[0], self.inner_size))
+        self.inner(pre, step, cache, inner, 1.0, write_cache)
+        return self.o.forward(inner, out_dtype=self.out_dtype)
+
+
+class CappedWindowAttention(Mixer):
+    """Softmax attention over a sliding window with a capped score, on heads whose queries and keys have unit mean square:
+
+        q = unit(rotate(W_q x))      k = unit(rotate(W_k x))      v = W_v x        unit(z) = z / sqrt(mean(z^2) + eps), per head
+            (rotation of the first rot_dims entries of a head in pairs of neighbours; no weight in the norm behind it)
+        the query at position i sees the keys j with 0 <= i - j < window (window 0: every j <= i)
+        out = softmax(softcap * tanh(q . k * scale / softcap)) v            (softcap 0: the scores as they are)
+
+    Values may have another size than keys.  W_q | W_k | W_v are one product with 32-bit output; one kernel rotates, norms
+    and writes keys and values into their pages.  Beside forward(), the mixer offers its steps apart (in_names / in_sizes,
+    inner, `o`)."""
+    recordable = True
+
+    def __init__(self, rt: Runtime, prefix: str, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
+                 softcap: float, position_encoding: Optional[NeighbourRotary], window: int, eps: float,
+                 out_dtype: Optional[torch.dtype] = None):
+        if heads % kv_heads:
+            raise ValueError(f"{heads} query heads are not a multiple of {kv_heads} kv heads")
+        if position_encoding is not None and not hasattr(position_encoding, "pair_table"):
+            raise ValueError("this attention rotates pairs of neighbours (pair_table)")
+        self.rt, self.prefix, self.width = rt, prefix, width
+        self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
+        self.scale, self.softcap, self.window, self.eps = float(scale), float(softcap), int(window), float(eps)
+        self.position_encoding, self.out_dtype = position_encoding, out_dtype
+        self.q_size, self.k_size, self.v_size, self.inner_size = heads * dim, kv_heads * dim, kv_heads * vdim, heads * vdim
+        self.proj = Linear(rt, self.in_names(), width, self.in_sizes())
+        self.o = Linear(rt, f"{prefix}.o", self.inner_size, width)
+
+    def in_names(self) -> list[str]:
+        return [f"{self.prefix}.q", f"{self.prefix}.k", f"{self.prefix}.v"]
+
+    def in_sizes(self) -> list[int]:
+        return [self.q_size, self.k_size, self.v_size]
+
+    def children(self) -> list[Part]:
+        return [self.proj, self.o]
+
+    def plan_key(self) -> Optional[Hashable]:
+        return _attention_plan_key(self.rt, self.heads, self.kv_heads, self.dim, self.vdim)
+
+    def plan(self, batch: BatchShape) -> Optional[StepPlan]:
+        return _attention_plan(batch, self.heads, self.kv_heads)
+
+    def cache_request(self) -> KVPages:
+        return KVPages(self.kv_heads, self.dim, self.window, v_head_dim=self.vdim if self.vdim != self.dim else 0)
+
+    def inner(self, pre: torch.Tensor, step: StepContext, cache: KVCacheView, out: torch.Tensor, out_scale: float = 1.0,
+              write_cache: bool = True) -> None:
+        """pre: float32 [T, >= sum(in_sizes())], the columns q | k | v of this mixer; out: [T, inner_size] in the activation
+        type (contiguous) receives the heads."""
+        if out_scale != 1.0 or not out.is_contiguous():
+            raise ops.KernelError("this attention writes unscaled heads into a matrix of their own")
+        rt = self.rt
+        T, H, G, D, V = pre.shape[0], self.heads, self.kv_heads, self.dim, self.vdim
+        c1, c2, c3 = self.q_size, self.q_size + self.k_size, self.q_size + self.k_size + self.v_size
+        inv_freq, rot = self.position_encoding.pair_table() if self.position_encoding is not None else (None, 0)
+        q = rt.empty((T, H, D))
+        ops.rope_kv(pre[:, :c1], pre[:, c1:c2], pre[:, c2:c3], q, step.positions, H, G if write_cache else 0, D, self.eps, rt.stream,
+                    inv_freq=inv_freq, rot_dim=rot, k_cache=cache.k, v_cache=cache.v, token_seq=step.token_seq,
+                    block_table=step.block_tables[cache.group], page_size=cache.page_size, v_dim=V, pairs=True, unit=True)
+        ops.attention(q, out.view(T, H, V), cache.k, cache.v, step, cache.group, H, G, D, cache.page_size, self.window, self.scale,
+                      rt.stream, plan=step.plans.get(self.plan_key()), v_dim=V if V != D else 0, softcap=self.softcap)
 
     def forward(self, h: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
         pre = self.proj.forward(h, out_dtype=torch.float32)

@@ -40,6 +40,7 @@ class ParamSpec:
     shape: tuple[int, ...]
     init: str = "linear"            # "linear" | "embedding" | "norm" | "unit": how random weights are drawn
     integer: bool = False           # integer tables are kept as int32
+    below: int = 0                  # integer tables: how random ones are drawn, rows of distinct numbers 0 .. below - 1 (0: any numbers)
 
 
 @dataclass(frozen=True)
@@ -146,6 +147,10 @@ class StepContext:
     span_hint: int = 0                          # bound on the context lengths to plan launches for (see BatchShape)
     # What the parts planned for this step, by their plan_key().
     plans: dict[Hashable, PlanView] = field(default_factory=dict)
+    token_ids: Optional[torch.Tensor] = None    # [T]; for parts that choose by the token itself
+    # What a part wants to keep for its later calls in the same run of the model (a block that runs several times may use
+    # again what depends on the tokens alone).  The model empties it before every run.
+    memo: dict[Hashable, Any] = field(default_factory=dict)
 
 
 @dataclass
@@ -171,6 +176,32 @@ class StreamCopy:
     copy in the kernel that adds a sublayer's output, so the next block of that kind need not make one; every other
     reader takes it for None."""
     x: torch.Tensor
+
+
+@dataclass
+class Pending:
+    """What is still to be added to the residual stream, handed on as `delta` for the norm that reads the stream next
+    (Norm.takes_pending): that norm adds it in its own pass over the row.
+
+        plain    up to two float32 matrices, added as they are
+        vector   one float32 row, added to every row
+        output   a sublayer's output that goes through `norm` (an RMSNorm) before it is added: a tensor, or ExpertSum"""
+    plain: tuple = ()
+    vector: Optional[torch.Tensor] = None
+    output: Any = None
+    norm: Any = None
+
+
+@dataclass
+class ExpertSum:
+    """The output of routed experts that is not summed yet: out[t] = sum_k weights[t, k] rows[place_of[t, k]] (+ the output
+    of the expert every token uses, times sigmoid(gate_weight . gate_input[t]) if there is a gate)."""
+    rows: torch.Tensor                           # [places, width] float32
+    place_of: torch.Tensor                       # [T * top] int32
+    weights: Any                                 # [T, top] float32, or one number
+    always: Optional[torch.Tensor] = None        # [T, width]
+    gate_input: Optional[torch.Tensor] = None    # [T, width]
+    gate_weight: Optional[torch.Tensor] = None   # [width] float32
 
 
 @dataclass
@@ -228,6 +259,8 @@ class Norm(Part):
     # True: add_forward() also takes a tuple of two tensors as `delta` and adds both (blocks whose sublayers run side
     # by side hand their outputs on unsummed).
     takes_delta_parts = False
+    # True: add_forward() also takes a Pending as `delta`.
+    takes_pending = False
 
     def add_forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], out_dtype: torch.dtype,
                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -278,6 +311,9 @@ class Mixer(Part):
 
 class FeedForward(Part):
     accepts_sink = False
+    # True: forward() takes the keyword `unsummed`; with it the part may return an ExpertSum instead of a tensor, for a
+    # reader that forms the sum in its own pass over the row (Pending.output).
+    offers_unsummed = False
 
     def row_scaled_ok(self, num_tokens: int) -> bool:
         return False
@@ -294,6 +330,7 @@ class Block(Part):
     offers_delta_parts = False
     takes_delta_parts = False       # True: forward() takes such a tuple as `delta` (its first norm adds both)
     takes_stream_copy = False       # True: forward() takes a StreamCopy as `delta` (see there)
+    takes_pending = False           # True: forward() takes a Pending as `delta`
 
     def cache_request(self) -> KVPages | StateSlot | None | tuple:
         """What a call of this block keeps of past tokens: the mixer's cache, unless the block has state of its own

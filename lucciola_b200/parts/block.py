@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 from .. import ops
-from .base import Block, FeedForward, Mixer, Norm, NormSink, Part, RowScaled, StepContext, StreamCopy
+from .base import Block, FeedForward, Mixer, Norm, NormSink, Part, Pending, RowScaled, StepContext, StreamCopy
 from .causal_taps import CausalTaps
 
 
@@ -167,3 +167,39 @@ class PostNormBlock(Block):
             b = self.feed_forward.forward(residual if exact else h, step)
             h = self.ffn_norm.add_normed(residual, (b,), (1.0,), self.residual_mult, copy_dtype)
         return residual, (None if exact else StreamCopy(h))
+
+
+class SandwichNormBlock(Block):
+    """A norm in front of and a norm behind every sublayer: r += norm1b(mixer(norm1(r))); r += norm2b(ffn(norm2(r))).  A block
+    may have no feed-forward.  All four are RMS norms.
+
+    Where a norm behind a sublayer meets the norm in front of the next, one kernel does both and the add between them
+    (Pending, RMSNorm.add_forward): behind the mixer inside the block, and behind the feed-forward in the first norm of
+    the block that follows, to which the block hands its output on as a Pending.  Routed experts leave their weighted sum
+    to that kernel too (FeedForward.offers_unsummed)."""
+    recordable = True
+    takes_pending = True
+
+    def __init__(self, mixer: Mixer, feed_forward: Optional[FeedForward], mixer_norm: Norm, mixer_out_norm: Norm,
+                 ffn_norm: Optional[Norm], ffn_out_norm: Optional[Norm], act_dtype: torch.dtype):
+        if (feed_forward is None) != (ffn_norm is None) or (ffn_norm is None) != (ffn_out_norm is None):
+            raise ValueError("a feed-forward and its two norms come together")
+        if not all(n is None or n.takes_pending for n in (mixer_norm, ffn_norm)):
+            raise ValueError("the norms in front of the sublayers must take what is still to be added (Norm.takes_pending)")
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.mixer_out_norm, self.ffn_norm, self.ffn_out_norm = mixer_norm, mixer_out_norm, ffn_norm, ffn_out_norm
+        self.act_dtype = act_dtype
+
+    def children(self) -> list[Part]:
+        return [p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.ffn_norm, self.feed_forward, self.ffn_out_norm)
+                if p is not None]
+
+    def forward(self, residual: torch.Tensor, delta, step: StepContext, cache, write_cache: bool = True):
+        h = self.mixer_norm.add_forward(residual, delta, self.act_dtype)
+        a = self.mixer.forward(h, step, cache, write_cache)
+        pending = Pending(output=a, norm=self.mixer_out_norm)
+        if self.feed_forward is None:
+            return residual, pending
+        h = self.ffn_norm.add_forward(residual, pending, self.act_dtype)
+        b = self.feed_forward.forward(h, step, unsummed=True) if self.feed_forward.offers_unsummed else self.feed_forward.forward(h, step)
+        return residual, Pending(output=b, norm=self.ffn_out_norm)

@@ -54,7 +54,7 @@ class TokenEmbedding(Part):
             self.sin_freq = (self.sinusoid_base ** (-2.0 * i / self.hidden_size)).to(self.weight.device).contiguous()
 
     def forward(self, token_ids: torch.Tensor, positions: torch.Tensor | None = None, copy: torch.Tensor | None = None) -> torch.Tensor:
-        """`copy` (float32 [T, hidden]) receives the output a second time, for a model that adds it to the stream again."""
+        """`copy` (float32 or the activation type, [T, hidden]) receives the output a second time, for a model that adds it to the stream again."""
         out = self.rt.empty((token_ids.shape[0], self.hidden_size), torch.float32)
         if copy is not None and self.sinusoid_base is not None:
             raise ValueError("no second copy of an embedding with sinusoidal positions")
@@ -77,9 +77,12 @@ class OutputHead(Part):
 
 
     def __init__(self, rt: Runtime, name: str, vocab_size: int, hidden_size: int, tied_to: TokenEmbedding | None,
-                 scale: float = 1.0):
+                 scale: float = 1.0, softcap: float = 0.0):
         self.rt, self.name, self.tied_to = rt, name, tied_to
         self.vocab_size = vocab_size
+        if softcap and scale != 1.0:
+            raise ValueError("logits are scaled or capped, not both")
+        self.softcap = float(softcap)       # > 0: logits become softcap * tanh(logits / softcap), in 32-bit in the product's epilogue
         self.scale = float(scale)           # the logits are multiplied by this, in 32-bit
         self.proj = Linear(rt, name, hidden_size, vocab_size)
 
@@ -97,7 +100,7 @@ class OutputHead(Part):
             self.proj.bind(get)
 
     def forward(self, h: torch.Tensor) -> torch.Tensor:
-        logits = self.proj.forward(h, out_dtype=torch.float32)
+        logits = self.proj.forward(h, out_dtype=torch.float32, post="cap" if self.softcap else None, post_c=self.softcap)
         if self.scale != 1.0:
             ops.scale_(logits, self.scale, self.rt.stream)
         return logits

@@ -78,15 +78,17 @@ class Linear(Part):
         """Whether forward() takes rows without their norm's factor: the tensor-core products apply it in their epilogues."""
         return self.rt.fast_kernels and self.in_features % 8 == 0
 
-    def forward(self, x, out_dtype: torch.dtype | None = None, rows: int | None = None) -> torch.Tensor:
-        """y = x . W^T; with `rows`, only the first `rows` output features.  x: a tensor, or RowScaled."""
+    def forward(self, x, out_dtype: torch.dtype | None = None, rows: int | None = None, post: str | None = None,
+                post_c: float = 0.0) -> torch.Tensor:
+        """y = post(x . W^T) (an element operation in the product's epilogue, see ops.POST_OPS); with `rows`, only the first
+        `rows` output features.  x: a tensor, or RowScaled."""
         M = x.shape[0]
         w = self.weight if rows is None else self.weight[:rows]
         y = self.rt.empty((M, w.shape[0]), out_dtype or self.rt.act_dtype)
         if isinstance(x, RowScaled):
             if not (self.row_scaled_ok(M) and ops.gemm_tcgen05_ok(y, x.x, w)):
                 raise ops.KernelError("this product was handed rows without their norm factor for sizes it cannot take them in")
-            ops.gemm_tcgen05(y, x.x, w, self.rt.stream, sumsq=x.sumsq, eps=x.eps)
+            ops.gemm_tcgen05(y, x.x, w, self.rt.stream, sumsq=x.sumsq, eps=x.eps, post=post, post_c=post_c)
             return y
-        ops.linear(y, x, w, self.rt.stream, fast=self.rt.fast_kernels)
+        ops.linear(y, x, w, self.rt.stream, fast=self.rt.fast_kernels, post=post, post_c=post_c)
         return y

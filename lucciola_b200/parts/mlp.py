@@ -81,7 +81,8 @@ class SwiGLUFeedForward(GatedFeedForward):
 
 
 class DenseFeedForward(FeedForward):
-    """A feed-forward without a gate: down( act(up(h)) ).  `act` is one of ops.PLAIN_ACTS ("relu2" is relu(z)^2); xIELU,
+    """A feed-forward without a gate: down( act(up(h)) ).  `act` is "gelu" (the exact form, in the up product's epilogue) or one
+    of ops.PLAIN_ACTS ("relu2" is relu(z)^2); xIELU,
 
         z > 0: softplus(p) z^2 + z / 2        z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2,
 
@@ -91,8 +92,8 @@ class DenseFeedForward(FeedForward):
 
     def __init__(self, rt: Runtime, up_name: str, down_name: str, hidden_size: int, intermediate_size: int, act: str = "xielu",
                  act_name: Optional[str] = None, out_dtype: Optional[torch.dtype] = None):
-        if act not in ops.PLAIN_ACTS:
-            raise ValueError(f"activation {act!r} of a dense feed-forward is not one of {sorted(ops.PLAIN_ACTS)}")
+        if act not in ops.PLAIN_ACTS and act != "gelu":
+            raise ValueError(f"activation {act!r} of a dense feed-forward is not one of {['gelu', *sorted(ops.PLAIN_ACTS)]}")
         if (act == "xielu") != (act_name is not None):
             raise ValueError("xielu, and only xielu, takes a tensor with its two numbers")
         self.rt, self.act, self.act_name, self.out_dtype = rt, act, act_name, out_dtype
@@ -115,6 +116,8 @@ class DenseFeedForward(FeedForward):
             self.p0, self.p1 = sp(p), 0.5 + sp(q)
 
     def forward(self, h, step: StepContext):
+        if self.act == "gelu":
+            return self.down.forward(self.up.forward(h, post="gelu"), out_dtype=self.out_dtype)
         u = self.up.forward(h)
         a = self.rt.empty(u.shape)
         ops.activation(a, u, self.act, self.rt.stream, self.p0, self.p1)

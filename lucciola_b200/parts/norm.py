@@ -4,6 +4,9 @@
 GroupRMSNorm cuts the row into equal consecutive parts with a root mean square each; with one group it is the
 same function (it does not offer itself as a sink of a product's epilogue, which forms one sum a row).
 
+RMSNorm.add_forward() also takes a Pending: the terms still to be added to the stream, of which one may go through another
+RMSNorm first (models that norm what a sublayer returns as well as what the next one reads); one kernel forms both norms.
+
 LayerNorm is the centred norm with a weight and no bias, y = (x - mean) / sqrt(var + eps) * w; it can also sit BEHIND a
 sublayer (add_normed), for blocks that norm what a sublayer returns."""
 from __future__ import annotations
@@ -13,7 +16,7 @@ from typing import Callable, Optional
 import torch
 
 from .. import ops
-from .base import Norm, NormSink, ParamSpec, Runtime
+from .base import ExpertSum, Norm, NormSink, ParamSpec, Pending, Runtime
 
 
 class RMSNorm(Norm):
@@ -36,11 +39,16 @@ class RMSNorm(Norm):
     def as_sink(self, residual: torch.Tensor) -> Optional[NormSink]:
         return NormSink(residual, self.weight, self.eps)
 
-    def add_forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], out_dtype: torch.dtype,
+    takes_pending = True
+
+    def add_forward(self, residual: torch.Tensor, delta, out_dtype: torch.dtype,
                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = self.rt.empty((n, self.size), out_dtype)
-        ops.add_rmsnorm(out, residual, delta, self.weight, self.eps, self.rt.stream, rows=rows)
+        if isinstance(delta, Pending):
+            ops.stream_norm(residual, self.rt.stream, out=out, weight=self.weight, eps=self.eps, rows=rows, **pending_terms(delta))
+        else:
+            ops.add_rmsnorm(out, residual, delta, self.weight, self.eps, self.rt.stream, rows=rows)
         return out
 
     def add_forward_pair(self, residual: torch.Tensor, deltas: tuple, other: Optional["RMSNorm"], out_dtype: torch.dtype):
@@ -54,6 +62,19 @@ class RMSNorm(Norm):
         ops.add_rmsnorm_pair(a, b, residual, tuple(deltas), self.weight, other.weight if other is not None else None, self.eps,
                              self.rt.stream)
         return a, b
+
+
+def pending_terms(p: Pending) -> dict:
+    """A Pending as keywords of ops.stream_norm."""
+    terms: dict = {"adds": p.plain, "vec": p.vector}
+    if p.output is not None:
+        terms.update(y_weight=p.norm.weight, y_eps=p.norm.eps)
+        if isinstance(p.output, ExpertSum):
+            o = p.output
+            terms["experts"] = (o.rows, o.place_of, o.weights, o.always, o.gate_input, o.gate_weight)
+        else:
+            terms["y"] = p.output
+    return terms
 
 
 class GroupRMSNorm(Norm):

@@ -29,6 +29,9 @@ def random_tensor(spec: ParamSpec, seed: int, std: float, norm_std: float, dtype
     device = torch.device(device)
     g = torch.Generator(device=device)
     g.manual_seed(_tensor_seed(seed, spec.name))
+    if spec.integer and spec.below:                # every row: distinct numbers below the bound
+        rank = torch.rand((*spec.shape[:-1], spec.below), generator=g, device=device)
+        return rank.argsort(dim=-1)[..., :spec.shape[-1]].to(torch.int32).contiguous()
     if spec.integer:
         return torch.randint(0, 2 ** 15, spec.shape, generator=g, device=device, dtype=torch.int32)
     if spec.init == "unit":                        # a bound or a rate that lies inside (0, 1)
