@@ -36,6 +36,9 @@ feed-forward), beside Bonolorn and Qwen3 at equal sizes.
 `--design venitar` does the same for the Venitar design (pre-norm blocks of which the first two run twice; window attention with
 YaRN rotation and a sigmoid gate beside a gated delta rule with a decay for every key channel, retention, and attention in chunks
 whose values are its keys, with a sink; a relu-squared feed-forward), beside Nelovik and Qwen3 at equal sizes.
+`--design nulalorn` does the same for the Nulalorn design (a norm in front of and behind every sublayer; two layers that run twice,
+each pass entered through a map of the stream and the embedding; window attention with capped scores on unit heads; gelu
+feed-forwards and experts named by a table of the token ids in turn), beside Bonolorn and Qwen3 at equal sizes.
 
 Peaks come from MEASURED_PEAKS.json beside this file when the driver wrote it, else from the
 fallback figures 6650 GB/s and 1590 TFLOP/s.  The timed work reads far more than the 126 MB of L2
@@ -444,7 +447,7 @@ DESIGN_SIZES = {
 
 # the models a --design run measures: the design and the nearest ones beside it
 DESIGN_BESIDE = {"riruzen": ("riruzen", "qwen3"), "bonolorn": ("riruzen", "qwen3", "bonolorn"), "nelovik": ("nelovik", "bonolorn", "qwen3"),
-                 "venitar": ("venitar", "nelovik", "qwen3")}
+                 "venitar": ("venitar", "nelovik", "qwen3"), "nulalorn": ("nulalorn", "bonolorn", "qwen3")}
 
 
 def design_configs(size: dict, layers: int, positions: int) -> dict:
@@ -499,7 +502,43 @@ def design_configs(size: dict, layers: int, positions: int) -> dict:
     venitar = {"architecture": "Venitar", "vocab": size["vocab"], "width": W, "embedding": {"scale": 2.0}, "norm": {"eps": 1e-6},
                "loop": {"start": 0, "stop": 2 if looped else 0, "times": 2 if looped else 1},
                "layers": [vorder[i % 4] for i in range(layers - 2 if looped else layers)]}
-    return {"riruzen": riruzen, "qwen3": qwen3, "bonolorn": bonolorn, "nelovik": nelovik, "venitar": venitar}
+    # Nulalorn: `layers` runs of layers, of which the second and third run twice (so two fewer distinct layers); all heads attend
+    # (a quarter as many kv heads, window 1024, cap 30, half of a head rotated with scaled frequencies); layers take a gelu
+    # feed-forward of the size's `ff` and 16 experts of `ff / 8` (4 a token by its id, one of `ff / 4` for every token) in turn
+    nmix = {"heads": H, "kv_heads": max(H // 4, 1), "dim": D, "vdim": D, "scale": 1.2 * D ** -0.5, "softcap": 30.0, "mask": {"size": 1024},
+            "rot": {"dims": D // 2, "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    nmoe = {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": size["ff"] // 8}, "shared": {"ff": size["ff"] // 4}}
+    nulalorn = {"architecture": "Nulalorn", "vocab": size["vocab"], "width": W, "norm": {"eps": 1e-6}, "logit_softcap": 50.0,
+                "layers": [{"type": "attention", "mixer": nmix, "mlp": ffd if i % 2 == 0 else nmoe} for i in range(layers - 2 if looped else layers)]}
+    if looped:
+        nulalorn["loop"] = {"start": 1, "stop": 3, "times": 2}
+    return {"riruzen": riruzen, "qwen3": qwen3, "bonolorn": bonolorn, "nelovik": nelovik, "venitar": venitar, "nulalorn": nulalorn}
+
+
+def nulalorn_costs(cfg: dict) -> dict:
+    """The same for a Nulalorn configuration, run by run (a layer that runs twice is read twice).  The window bounds the keys and
+    values a decoded token reads; of the experts a step of B tokens reads at most B * top a run (`expert_layers`).  A pass is
+    entered through a [width, 2 width] map whose half for the embedding's output is read once a step."""
+    W = cfg["width"]
+    loop = cfg.get("loop") or {"start": 0, "stop": 0, "times": 0}
+    runs = list(range(loop["start"])) + list(range(loop["start"], loop["stop"])) * loop["times"] + list(range(loop["stop"], len(cfg["layers"])))
+    weights = W * W * (loop["times"] + 1) if loop["stop"] > loop["start"] else 0
+    active = 0
+    attn, cache, expert_layers = [], [], []
+    for i in runs:
+        a, f = cfg["layers"][i]["mixer"], cfg["layers"][i]["mlp"]
+        weights += (a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"])) * W + W * a["heads"] * a["vdim"]
+        cache.append(lambda c, a=a: 2 * a["kv_heads"] * (a["dim"] + a["vdim"]) * min(c, a["mask"]["size"]))
+        attn.append(lambda T, a=a: a["heads"] * 2.0 * (a["dim"] + a["vdim"]) * sum(min(t + 1, a["mask"]["size"]) for t in range(T)))
+        if f["kind"] == "dense":
+            weights += 2 * f["ff"] * W
+        else:
+            weights += 2 * f["shared"]["ff"] * W
+            one = 2 * f["expert"]["ff"] * W
+            expert_layers.append((one, f["router"]["experts"], f["router"]["top"]))
+            active += f["router"]["top"] * one
+    return {"weight_bytes": 2 * (weights + cfg["vocab"] * W), "token_bytes": 0, "request_bytes": 0, "flops_per_token": 2.0 * (weights + active),
+            "attn_flops": lambda T: sum(f(T) for f in attn), "cache_bytes": lambda c: sum(f(int(c)) for f in cache), "expert_layers": expert_layers}
 
 
 def venitar_costs(cfg: dict) -> dict:
@@ -608,6 +647,8 @@ def design_costs(name: str, cfg: dict) -> dict:
         return nelovik_costs(cfg)
     if name == "venitar":
         return venitar_costs(cfg)
+    if name == "nulalorn":
+        return nulalorn_costs(cfg)
     if name == "qwen3":
         L = cfg["num_hidden_layers"]
         per_layer, weight_bytes, kv = model_bytes_and_flops(cfg, L)
@@ -666,7 +707,7 @@ def run_design(args) -> int:
             pages = 64 * (-(-(ctx + K + Wm + 8) // page)) + -(-T // page) + 64
             options = EngineOptions(dtype="bfloat16", block_size=page, max_blocks=pages, max_num_seqs=66, max_tokens_per_step=T + 64,
                                     use_cuda_graph=not (args.no_graph or args.profile))
-            if args.design == "venitar":
+            if args.design in ("venitar", "nulalorn"):
                 # designs whose positions have no limit of their own get the run's: block tables as wide as the run needs
                 options = EngineOptions(dtype="bfloat16", block_size=page, max_blocks=pages, max_num_seqs=66, max_tokens_per_step=T + 64,
                                         use_cuda_graph=not (args.no_graph or args.profile), max_model_len=max(ctx, T) + K + Wm + 64)
@@ -773,12 +814,12 @@ def main() -> int:
     ap.add_argument("--portion", type=int, default=512, help="tokens of the portion of a --profile mixed step")
     ap.add_argument("--time-kernel", choices=["attention_key_ranges"], default=None,
                     help="time one kernel alone over a grid of sizes, print a line of JSON a case, and exit")
-    ap.add_argument("--design", choices=["riruzen", "bonolorn", "nelovik", "venitar"], default=None,
+    ap.add_argument("--design", choices=["riruzen", "bonolorn", "nelovik", "venitar", "nulalorn"], default=None,
                     help="instead of the default workload: prefill and decode of this design beside the Qwen3 decoder at equal "
                          "sizes (--design-sizes; --layers, default 8; --prefill-tokens; --context up to 2048; --profile decode|prefill "
                          "with --batch runs one step between cudaProfilerStart/Stop)")
     ap.add_argument("--design-sizes", default="w2048,w4096", help="which of %s" % ", ".join(sorted(DESIGN_SIZES)))
-    ap.add_argument("--design-models", default="", help="which of riruzen, qwen3, bonolorn, nelovik, venitar (empty: the design and those beside it)")
+    ap.add_argument("--design-models", default="", help="which of riruzen, qwen3, bonolorn, nelovik, venitar, nulalorn (empty: the design and those beside it)")
     args = ap.parse_args()
     if args.time_kernel == "attention_key_ranges":
         return time_attention_key_ranges()
