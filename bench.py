@@ -511,7 +511,7 @@ def design_configs(size: dict, layers: int, positions: int) -> dict:
     nulalorn = {"architecture": "Nulalorn", "vocab": size["vocab"], "width": W, "norm": {"eps": 1e-6}, "logit_softcap": 50.0,
                 "layers": [{"type": "attention", "mixer": nmix, "mlp": ffd if i % 2 == 0 else nmoe} for i in range(layers - 2 if looped else layers)]}
     if looped:
-        nulalorn["loop"] = {"start": 1, "stop": 3, "times": 2}
+        nulalorn["loop"] = {"start": 1, "stop": 3, "times": 2} if layers > 4 else {"start": 0, "stop": 2, "times": 2}
     return {"riruzen": riruzen, "qwen3": qwen3, "bonolorn": bonolorn, "nelovik": nelovik, "venitar": venitar, "nulalorn": nulalorn}
 
 
