@@ -69,6 +69,8 @@ struct TcAttnParams {
   float scale_log2;
   float cap_raw, cap_exp;                   // cap_raw > 0: raw score s <- cap_raw * tanh(s / cap_raw), cap_raw = softcap / scale,
                                             // cap_exp = 2 log2(e) / cap_raw
+  int cap_terms;                            // > 0 (5 or 7): raw scores have a known bound and the capped score, in powers of two and
+  float cap_coef[7];                        // with the scale in it, is s * sum_i cap_coef[i] s^(2i); no distance bias then
   const float* slopes;                      // optional [num_q_heads]: the score of key j for the query at position i is lowered by
   float inv_scale;                          // slopes[h] * (i - j); 1 / scale brings that into the raw score's units
   // With gridDim.z > 1 the keys of every work item are cut into gridDim.z ranges of whole blocks, one CTA each; a CTA
@@ -194,6 +196,7 @@ __device__ __forceinline__ void ta_unpack2(uint64_t v, float& a, float& b) { asm
 __device__ __forceinline__ uint64_t ta_fma2(uint64_t a, uint64_t b, uint64_t c) {
   uint64_t d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d;
 }
+__device__ __forceinline__ uint64_t ta_mul2(uint64_t a, uint64_t b) { uint64_t d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
 __device__ __forceinline__ uint64_t ta_add2(uint64_t a, uint64_t b) { uint64_t d; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
 __device__ __forceinline__ float ta_max3(float a, float b, float c) { float d; asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c)); return d; }
 // Which wait gave up (what lb_attention_tcgen05_device_error reports).
@@ -430,7 +433,11 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
     const int row_lo = p.window > 0 ? max(0, row_pos - p.window + 1) : 0;
     const float row_bias = (p.slopes && row_valid) ? p.slopes[kvh * G + r % G] * p.inv_scale : 0.f;   // this row's head: its distance slope
     const int tile_pos0 = pos0 + t * per;                    // the smallest position among the tile's rows
-    float m_ref = -INFINITY, l_run = 0.f;
+    const int tile_lo = p.window > 0 ? tile_pos0 + per - p.window : 0;      // from here on every row's window has begun
+    // Capped scores with a known bound need no running maximum: 2^score stays far inside the range of a float whatever the
+    // keys are, so the reference is 0 throughout and O is never rescaled.
+    const bool bounded = p.cap_terms > 0;
+    float m_ref = bounded ? 0.f : -INFINITY, l_run = 0.f;
     bool ok = true;
 
     for (int i = 0; i < nblocks; ++i) {
@@ -439,7 +446,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
       ok = ta_mbar_wait(s_full(t, b), (uint32_t)((i >> 1) & 1), abort_flag, TA_ERR_S_FULL);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const bool need_mask = (kb + TA_KEYS - 1 > tile_pos0) || (p.window > 0) || (kb < lo_tile) || (kb + TA_KEYS > kend);
+      const bool need_mask = (kb + TA_KEYS - 1 > tile_pos0) || (kb < tile_lo) || (kb < lo_tile) || (kb + TA_KEYS > kend);
       float x[TA_KEYS];
       {
         uint32_t v[64];
@@ -447,7 +454,31 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
 #pragma unroll
         for (int j = 0; j < 64; ++j) x[j] = __uint_as_float(v[j]);
       }
-      if (p.cap_raw > 0.f) {
+      if (bounded) {
+        // the cap as an odd polynomial, two keys an instruction, straight to the exponents
+        uint64_t c[7];
+#pragma unroll
+        for (int i = 0; i < 7; ++i) c[i] = ta_pack2(p.cap_coef[i], p.cap_coef[i]);
+        if (p.cap_terms <= 5) {
+#pragma unroll
+          for (int j = 0; j < TA_KEYS; j += 2) {
+            const uint64_t s2 = ta_pack2(x[j], x[j + 1]), t2 = ta_mul2(s2, s2);
+            uint64_t q = ta_fma2(c[4], t2, c[3]);
+#pragma unroll
+            for (int i = 2; i >= 0; --i) q = ta_fma2(q, t2, c[i]);
+            ta_unpack2(ta_mul2(s2, q), x[j], x[j + 1]);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < TA_KEYS; j += 2) {
+            const uint64_t s2 = ta_pack2(x[j], x[j + 1]), t2 = ta_mul2(s2, s2);
+            uint64_t q = ta_fma2(c[6], t2, c[5]);
+#pragma unroll
+            for (int i = 4; i >= 0; --i) q = ta_fma2(q, t2, c[i]);
+            ta_unpack2(ta_mul2(s2, q), x[j], x[j + 1]);
+          }
+        }
+      } else if (p.cap_raw > 0.f) {
 #pragma unroll
         for (int j = 0; j < TA_KEYS; ++j) x[j] = capped_score(x[j], p.cap_raw, p.cap_exp);
       }
@@ -463,6 +494,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
           if (key > row_pos || key < row_lo) x[j] = -INFINITY;
         }
       }
+      if (!bounded) {
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains of three-input maxima
 #pragma unroll
       for (int j = 0; j < TA_KEYS; j += 8) {
@@ -496,6 +528,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
           ta_tmem_wait_st();
         }
       }
+      }
       const float m_use = m_ref == -INFINITY ? 0.f : m_ref;
       // p = 2^(s * scale - m), the row's sum, P (two keys a column) over the first 32 columns of this S buffer.
       // Pairs of keys in packed instructions.  (Tried: a cubic for 2^f on the FMA pipe for half or a quarter of the
@@ -506,8 +539,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, TcAttnParams
       uint32_t w[32];
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
-        float y0, y1;
-        ta_unpack2(ta_fma2(ta_pack2(x[2 * j], x[2 * j + 1]), scale2, negm2), y0, y1);
+        float y0 = x[2 * j], y1 = x[2 * j + 1];
+        if (!bounded) ta_unpack2(ta_fma2(ta_pack2(y0, y1), scale2, negm2), y0, y1);
         const float p0 = exp2_approx(y0), p1 = exp2_approx(y1);          // 2^-inf = 0 for masked keys
         sum2 = ta_add2(sum2, ta_pack2(p0, p1));
         __nv_bfloat162 b2 = __floats2bfloat162_rn(p0, p1);
@@ -685,7 +718,10 @@ LB_EXPORT int lb_attention_tcgen05(const void* q, void* out, const void* k_cache
                                    const int* block_table, const void* tiles, int num_tiles, int num_tokens,
                                    int num_q_heads, int num_kv_heads, int head_dim, int page_size, int num_pages,
                                    int max_pages, int window, float scale, int key_splits, float* workspace,
-                                   long long workspace_elems, const float* slopes, float softcap, cudaStream_t stream) {
+                                   long long workspace_elems, const float* slopes, float softcap, int cap_terms,
+                                   const float* cap_coef, cudaStream_t stream) {
+  LB_CHECK_ARG(cap_terms >= 0 && cap_terms <= 7 && (cap_terms == 0 || (cap_coef && softcap > 0.f && !slopes)),
+               "attention_tcgen05: a polynomial of %d terms stands for a cap, without a distance bias", cap_terms);
   LB_CHECK_ARG(softcap >= 0.f && (softcap == 0.f || scale > 0.f), "attention_tcgen05: a cap of %f needs a positive scale", (double)softcap);
   LB_CHECK_ARG(slopes == nullptr || scale > 0.f, "attention_tcgen05: a distance bias needs a positive scale");
   LB_CHECK_ARG(lb_attention_tcgen05_ok(num_q_heads, num_kv_heads, head_dim, page_size),
@@ -715,6 +751,8 @@ LB_EXPORT int lb_attention_tcgen05(const void* q, void* out, const void* k_cache
   p.tiles = (const int4*)tiles; p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.group = group;
   p.page_size = page_size; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
   p.slopes = slopes; p.inv_scale = slopes ? 1.f / scale : 0.f;
+  p.cap_terms = cap_terms;
+  for (int i = 0; i < 7; ++i) p.cap_coef[i] = i < cap_terms ? cap_coef[i] : 0.f;
   p.cap_raw = softcap > 0.f ? softcap / scale : 0.f; p.cap_exp = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   p.page_shift = 0;
   while ((1 << p.page_shift) < page_size) ++p.page_shift;

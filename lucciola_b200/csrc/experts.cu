@@ -299,11 +299,15 @@ __global__ void __launch_bounds__(256) expert_gemm_plain_kernel(ExpertGemmParams
 }
 
 // tensor cores (mma.sync m16n8k16), bfloat16 operands, 32-bit sums: a tile of 64 places x 128 output columns a CTA of
-// eight warps (warp w: rows (w & 1) * 32 .., columns (w >> 1) * 32 ..); K in blocks of 32 through four stages of shared
+// eight warps (warp w: rows (w & 1) * 32 .., columns (w >> 1) * 32 ..); K in blocks of 64 through four stages of shared
 // memory that 16-byte asynchronous copies fill three blocks ahead of the tensor cores (with a few tokens the kernel
 // streams the experts' weights, and the copies in flight are what fills the memory pipe); fragments by ldmatrix from
-// rows padded to 80 bytes.  K a multiple of 8, 16-byte aligned rows.
-constexpr int EM_BM = 64, EM_BK = 32, EM_LD = EM_BK + 8, EM_STAGES = 4;
+// rows padded to 144 bytes.  Rows of the tile that hold no place are zeros from the start and are neither fetched nor, by
+// 32, multiplied.  K a multiple of 8, 16-byte aligned rows.
+constexpr int EM_BM = 64, EM_STAGES = 4;
+// (gated tiles of 128 columns take K by 32, rows padded to 80 bytes, so that two CTAs still share an SM)
+template <bool GATED, int BN>
+__host__ __device__ constexpr int expert_mma_bk() { return GATED && BN == 128 ? 32 : 64; }
 
 __device__ __forceinline__ void ex_mma_16816(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -320,13 +324,13 @@ __device__ __forceinline__ void ex_cp_async16(void* dst, const void* src, bool v
 }
 
 template <bool GATED, int BN>
-constexpr int expert_mma_smem() { return EM_STAGES * (EM_BM + (GATED ? 2 : 1) * BN) * EM_LD * 2; }
+constexpr int expert_mma_smem() { return EM_STAGES * (EM_BM + (GATED ? 2 : 1) * BN) * (expert_mma_bk<GATED, BN>() + 8) * 2; }
 
 // BN: output columns of a tile, 128 or 64 (with few places a launch is a stream of weights, and narrower tiles are more
 // CTAs to share it out over the SMs)
 template <typename TY, bool GATED, int BN>
 __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p) {
-  constexpr int EM_BN = BN;
+  constexpr int EM_BN = BN, EM_BK = expert_mma_bk<GATED, BN>(), EM_LD = EM_BK + 8;
   constexpr int NW = BN / 32;                                     // blocks of 8 columns a warp: 4 or 2
   extern __shared__ __align__(16) uint8_t ex_smem[];
   constexpr int NB = GATED ? 2 : 1;
@@ -350,13 +354,23 @@ __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p
     src_row[tid] = place < r1 ? (p.gather ? p.pair_at[place] / p.top : place) : -1;
   }
   __syncthreads();
-  const int a_r = tid >> 2, a_c = (tid & 3) * 8;                  // this thread's piece of A: 64 rows x 4 pieces
-  const int a_row = src_row[a_r];
-  auto load_stage = [&](int st, int k0) {
-    ex_cp_async16(As + (st * EM_BM + a_r) * EM_LD + a_c, a_row >= 0 ? x + (size_t)a_row * p.ldx + k0 + a_c : x, a_row >= 0 && k0 + a_c < p.K);
+  constexpr int PIECES = EM_BK / 8;                               // 16-byte pieces of a row of a stage
+  const int c_r = tid / PIECES, c_c = (tid % PIECES) * 8;         // this thread's piece, the same in every 256 / PIECES rows
+  constexpr int R_STEP = 256 / PIECES;
+  int a_row[EM_BM / R_STEP];
 #pragma unroll
-    for (int it = 0; it < BN / 64; ++it) {
-      const int idx = tid + it * 256, r = idx >> 2, c = (idx & 3) * 8;   // BN rows x 4 pieces
+  for (int it = 0; it < EM_BM / R_STEP; ++it) a_row[it] = src_row[c_r + it * R_STEP];
+  for (int i = tid; i < EM_STAGES * EM_BM * EM_LD / 8; i += 256) reinterpret_cast<uint4*>(As)[i] = make_uint4(0u, 0u, 0u, 0u);
+  __syncthreads();
+  const bool warp_rows = r0 + wm < r1;                            // whether any of this warp's rows holds a place
+  auto load_stage = [&](int st, int k0) {
+#pragma unroll
+    for (int it = 0; it < EM_BM / R_STEP; ++it)
+      if (a_row[it] >= 0)
+        ex_cp_async16(As + (st * EM_BM + c_r + it * R_STEP) * EM_LD + c_c, k0 + c_c < p.K ? x + (size_t)a_row[it] * p.ldx + k0 + c_c : x, k0 + c_c < p.K);
+#pragma unroll
+    for (int it = 0; it < BN / R_STEP; ++it) {
+      const int r = c_r + it * R_STEP, c = c_c;
       const bool ok = n0 + r < ncols && k0 + c < p.K;
       int gr = n0 + r, ur = n0 + r;
       if (GATED) gate_up_rows(p, n0 + r, ncols, gr, ur);
@@ -387,6 +401,7 @@ __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p
     __syncthreads();                                                           // and the stage of block kb - 1 is free
     if (kb + EM_STAGES - 1 < nk) load_stage((kb + EM_STAGES - 1) % EM_STAGES, (kb + EM_STAGES - 1) * EM_BK);
     asm volatile("cp.async.commit_group;" ::: "memory");
+    if (!warp_rows) continue;
 #pragma unroll
     for (int kk = 0; kk < EM_BK; kk += 16) {
       uint32_t a[2][4];

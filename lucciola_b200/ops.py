@@ -110,7 +110,8 @@ _SIGNATURES = {
                               c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p,
                               c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lb_attention_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_float, c_void_p],
+                             c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_float, c_int, c_void_p,
+                             c_void_p],
     "lb_sample": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
 }
 
@@ -1232,13 +1233,43 @@ def attention_tcgen05_splits(num_tiles: int, num_kv_heads: int, max_span: int, s
     return best
 
 
+_cap_polynomials: dict = {}
+
+
+def cap_polynomial(scale: float, softcap: float, bound: float) -> list[float] | None:
+    """log2(e) softcap tanh(s scale / softcap) as s * sum_i c_i s^(2i) for raw scores |s| <= bound: Chebyshev interpolation of
+    the even factor, in 64-bit, with 5 or 7 terms; None if 7 do not reach an error of 2^-22 of the factor, or if the capped
+    scores reach so far that 2^score needs a reference to stay in a float's range."""
+    import numpy as np
+    key = (scale, softcap, bound)
+    if key not in _cap_polynomials:
+        b = bound * scale / softcap
+        value = lambda t: np.where(t > 0, np.tanh(b * np.sqrt(np.maximum(t, 1e-30))) / np.sqrt(np.maximum(t, 1e-30)), b)
+        found = None
+        if 0 < b <= 2.0 and softcap * np.tanh(b) * np.log2(np.e) <= 60.0:
+            at = np.linspace(0.0, 1.0, 2001)
+            for terms in (5, 7):
+                fit = np.polynomial.chebyshev.Chebyshev.interpolate(value, terms - 1, domain=[0.0, 1.0])
+                if np.max(np.abs(fit(at) / value(at) - 1.0)) <= 2.0 ** -22:
+                    a = fit.convert(kind=np.polynomial.Polynomial).coef
+                    a = np.concatenate([a, np.zeros(terms - len(a))])
+                    found = [float(np.log2(np.e) * softcap / bound * a[i] / bound ** (2 * i)) for i in range(terms)]
+                    break
+        _cap_polynomials[key] = found
+    return _cap_polynomials[key]
+
+
 def attention_tcgen05(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                       positions: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor, num_q_heads: int,
                       num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float, stream: int,
-                      key_splits: int = 1, slopes: torch.Tensor | None = None, softcap: float = 0.0) -> None:
+                      key_splits: int = 1, slopes: torch.Tensor | None = None, softcap: float = 0.0,
+                      score_bound: float = 0.0) -> None:
     """Attention of portions of prompts on tcgen05 (S and O in tensor memory).  tiles: int32 [n, 4] of
     (first token, tokens, request index, 0) with tokens <= 2 * (128 // (nq // nkv)).  With key_splits > 1 the keys of
-    every tile are cut into that many ranges, a CTA each, combined by a second kernel."""
+    every tile are cut into that many ranges, a CTA each, combined by a second kernel.
+    `score_bound` > 0 with a cap: no |q . k| is larger (queries and keys of unit mean square, say); the kernel may then form
+    the cap as a polynomial and leave the running maximum out."""
+    coef = cap_polynomial(scale, softcap, score_bound) if softcap > 0 and score_bound > 0 and slopes is None else None
     _check(q, "q", torch.bfloat16); _check(out, "attention output", torch.bfloat16)
     _check(k_cache, "k pool", torch.bfloat16); _check(v_cache, "v pool", torch.bfloat16)
     _check(positions, "positions", torch.int32); _check(block_table, "block table", torch.int32)
@@ -1250,21 +1281,21 @@ def attention_tcgen05(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
     _call("lb_attention_tcgen05", q.data_ptr(), out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
           positions.data_ptr(), block_table.data_ptr(), tiles.data_ptr(), tiles.shape[0], q.shape[0], num_q_heads,
           num_kv_heads, head_dim, page_size, k_cache.shape[0], block_table.shape[1], window, scale, key_splits,
-          _ptr(ws), ws_elems, _ptr(slopes), float(softcap), stream)
+          _ptr(ws), ws_elems, _ptr(slopes), float(softcap), len(coef) if coef else 0, (c_float * 7)(*coef) if coef else None, stream)
 
 
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step, group: int,
               num_q_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float,
               stream: int, plan=None, kv_share: int = 1, v_dim: int = 0, slopes: torch.Tensor | None = None,
               softcap: float = 0.0, sinks: torch.Tensor | None = None, pool: int = 0, pool_k: torch.Tensor | None = None,
-              pool_v: torch.Tensor | None = None, pool_group: int = -1, chunk: int = 0) -> None:
+              pool_v: torch.Tensor | None = None, pool_group: int = -1, chunk: int = 0, score_bound: float = 0.0) -> None:
     """Causal attention of this step's queries over the pages of their requests.  With a `plan` (tile lists
     by kind on the device, see parts/attention.py) the tensor-core kernels run where their conditions hold:
     portions of prompts go to the tcgen05 kernel, the rest (decoded tokens, short portions, other head
     sizes) to the mma.sync kernels; everything else, and every step without a plan, goes to the plain kernel.
     `kv_share` > 1: the plan's lists other than "big" were made for groups of num_q_heads / (num_kv_heads * kv_share)
     query heads, kv_share of which read one cached head (see attention_flash).  A capped score (`softcap`) is taken by
-    all of them, values of another size than the keys by all but the tcgen05 kernel.  Sinks and
+    all of them (`score_bound`: see attention_tcgen05), values of another size than the keys by all but the tcgen05 kernel.  Sinks and
     pooled blocks behind the window (`pool` tokens a block, their means in pool_k / pool_v, pages of group `pool_group`)
     and chunks (`chunk` = C: a query sees the keys of its own run of C positions only) run in the mma.sync kernel with
     16-byte copies, for portions and for decoded tokens, or in the plain kernel."""
@@ -1291,7 +1322,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
                                                              step.block_tables[group].shape[1]):
         attention_tcgen05(q, out, k_cache, v_cache, step.positions, step.block_tables[group], meta["big"],
                           num_q_heads, num_kv_heads, head_dim, page_size, window, scale, stream,
-                          key_splits=attention_tcgen05_splits(meta["big"].shape[0], num_kv_heads, span), slopes=slopes, softcap=softcap)
+                          key_splits=attention_tcgen05_splits(meta["big"].shape[0], num_kv_heads, span), slopes=slopes, softcap=softcap,
+                          score_bound=score_bound)
         kinds = ["rest"] if "rest" in meta else []
     for kind in kinds:
         tiles = meta[kind]

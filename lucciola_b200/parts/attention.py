@@ -642,7 +642,8 @@ class CappedWindowAttention(Mixer):
                     inv_freq=inv_freq, rot_dim=rot, k_cache=cache.k, v_cache=cache.v, token_seq=step.token_seq,
                     block_table=step.block_tables[cache.group], page_size=cache.page_size, v_dim=V, pairs=True, unit=True)
         ops.attention(q, out.view(T, H, V), cache.k, cache.v, step, cache.group, H, G, D, cache.page_size, self.window, self.scale,
-                      rt.stream, plan=step.plans.get(self.plan_key()), v_dim=V if V != D else 0, softcap=self.softcap)
+                      rt.stream, plan=step.plans.get(self.plan_key()), v_dim=V if V != D else 0, softcap=self.softcap,
+                      score_bound=1.02 * D)           # |q| and |k| are at most sqrt(D), but for their rounding to 16 bits
 
     def forward(self, h: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
         pre = self.proj.forward(h, out_dtype=torch.float32)

@@ -375,6 +375,54 @@ def test_a_query_finds_its_one_key_at_every_edge(dtype, heads, kv, dim, vdim, pa
     assert ops.device_error() == 0
 
 
+@pytest.mark.parametrize("scale,cap,terms", [(0.1, 30.0, 5), (0.12, 20.0, 7), (0.09, 12.0, 7), (0.2, 10.0, 0), (0.9, 90.0, 0)])
+@pytest.mark.parametrize("heads,kv,window", [(4, 2, 33), (8, 1, 100), (2, 2, 0)])
+def test_capped_scores_with_a_known_bound(scale, cap, terms, heads, kv, window):
+    """Heads of unit mean square: the cap as a polynomial without a running maximum where the bound allows it, and the
+    ordinary way where it does not, agree with a plain softmax; the key that equals the query stands at the bound itself, inside
+    the window, at its first place and at the place before it."""
+    from lucciola_b200 import ops
+    from lucciola_b200.parts.attention import plan_tiles
+    from lucciola_b200.parts.base import BatchShape
+    D, page, n, T = 128, 16, 330, 200
+    coef = ops.cap_polynomial(scale, cap, 1.02 * D)
+    assert (len(coef) if coef else 0) == terms
+    if coef:
+        s = torch.linspace(-D, D, 5001, dtype=torch.float64)
+        got = s * sum(c * s ** (2 * i) for i, c in enumerate(coef))
+        assert (got - cap * torch.tanh(s * scale / cap) / torch.log(torch.tensor(2.0, dtype=torch.float64))).abs().max() <= 1e-5
+    g = torch.Generator(device=DEV).manual_seed(heads)
+    unit = lambda x: x / x.pow(2).mean(-1, keepdim=True).sqrt()
+    per = heads // kv
+    table = torch.randperm(-(-n // page), generator=g, device=DEV).to(torch.int32).reshape(1, -1)
+    for back in (0, 1, max(window - 1, 5), window or 50):
+        q, K, V = unit(torch.randn(T, heads, D, device=DEV, generator=g)), unit(torch.randn(n, kv, D, device=DEV, generator=g)), torch.randn(n, kv, D, device=DEV, generator=g)
+        for t in range(0, T, 37):
+            K[n - T + t - back] = q[t].reshape(kv, per, D)[:, 0] * (1.0 if t % 2 else -1.0)
+        kc = torch.full((table.shape[1], kv, page, D), float("nan"), dtype=torch.bfloat16, device=DEV)
+        vc = kc.clone()
+        pos = torch.arange(n, device=DEV)
+        kc[table[0, pos // page].long(), :, pos % page] = K.to(torch.bfloat16)
+        vc[table[0, pos // page].long(), :, pos % page] = V.to(torch.bfloat16)
+        qb, Kd, Vd = q.to(torch.bfloat16), K.to(torch.bfloat16).double(), V.to(torch.bfloat16).double()
+        step = batch_of([T], [n - T])
+        made = plan_tiles(BatchShape([T], [n - T], T, n, n), per)
+        tiles = torch.from_numpy(made.arrays["big"]).to(DEV)
+        i = torch.arange(n - T, n, device=DEV)[:, None]
+        j = torch.arange(n, device=DEV)[None]
+        seen = (j <= i) & ((j > i - window) if window else (j >= 0))
+        want = torch.zeros(T, heads, D, dtype=torch.float64, device=DEV)
+        for h in range(heads):
+            s = plain.cap(qb[:, h].double() @ Kd[:, h // per].T * scale, cap).masked_fill(~seen, float("-inf"))
+            want[:, h] = torch.softmax(s, dim=-1) @ Vd[:, h // per]
+        for splits in (1, 3):
+            out = torch.full((T, heads, D), float("nan"), dtype=torch.bfloat16, device=DEV)
+            ops.attention_tcgen05(qb, out, kc, vc, step.positions, table, tiles, heads, kv, D, page, window, scale, stream(), key_splits=splits,
+                                  softcap=cap, score_bound=1.02 * D)
+            close(out, want, torch.bfloat16, rounded=1.2e-2)
+    assert ops.device_error() == 0
+
+
 # ---- the whole model -------------------------------------------------------------------------------------------------
 @pytest.fixture(scope="module")
 def models(tmp_path_factory):
