@@ -443,6 +443,83 @@ __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p
       }
 }
 
+// The same without a gate for steps with a few pairs an expert, on row tiles of at most 16 places (the dispatch is told so): the
+// launch is a stream of weights, so nearly all shared memory holds stages of weights, six of them in flight.  A CTA of four
+// warps takes 64 output columns, a warp 16.  Sums in the order of the kernel above.
+constexpr int EF_BM = 16, EF_BN = 64, EF_BK = 64, EF_LD = EF_BK + 8, EF_STAGES = 6;
+constexpr int EF_SMEM = EF_STAGES * (EF_BM + EF_BN) * EF_LD * 2;
+
+template <typename TY>
+__global__ void __launch_bounds__(128) expert_gemm_few_kernel(ExpertGemmParams p) {
+  extern __shared__ __align__(16) uint8_t ex_smem[];
+  bf16* As = reinterpret_cast<bf16*>(ex_smem);                    // [stage][BM][LD]
+  bf16* Bs = As + EF_STAGES * EF_BM * EF_LD;                      // [stage][BN][LD]
+  pdl_trigger();
+  pdl_wait();
+  if ((int)blockIdx.y >= p.meta[0]) return;
+  const int* m = p.meta + 4 + 3 * blockIdx.y;
+  const int e = m[0], r0 = m[1], r1 = min(m[2], m[1] + EF_BM);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n0 = blockIdx.x * EF_BN, wn = warp * 16;
+  const bf16* x = (const bf16*)p.x;
+  const bf16* w = (const bf16*)p.w + (size_t)e * p.N * p.K;
+  const int c_r = tid >> 3, c_c = (tid & 7) * 8;                  // this thread's row of A, and of every 16 rows of B; its 16-byte piece
+  const int place = r0 + c_r;
+  const int a_row = place < r1 ? (p.gather ? p.pair_at[place] / p.top : place) : -1;
+  auto load_stage = [&](int st, int k0) {
+    const bool k_ok = k0 + c_c < p.K;
+    ex_cp_async16(As + (st * EF_BM + c_r) * EF_LD + c_c, a_row >= 0 && k_ok ? x + (size_t)a_row * p.ldx + k0 + c_c : x, a_row >= 0 && k_ok);
+#pragma unroll
+    for (int it = 0; it < EF_BN / 16; ++it) {
+      const int r = c_r + it * 16;
+      const bool ok = k_ok && n0 + r < p.N;
+      ex_cp_async16(Bs + (st * EF_BN + r) * EF_LD + c_c, ok ? w + (size_t)(n0 + r) * p.K + k0 + c_c : w, ok);
+    }
+  };
+  float acc[2][4];
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int k = 0; k < 4; ++k) acc[j][k] = 0.f;
+  const int nk = (p.K + EF_BK - 1) / EF_BK;
+#pragma unroll
+  for (int st = 0; st < EF_STAGES - 1; ++st) {
+    if (st < nk) load_stage(st, st * EF_BK);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  const int a_lr = (lane & 7) + ((lane >> 3) & 1) * 8, a_lk = (lane >> 4) * 8;
+  const int b_lr = (lane & 7) + (lane >> 4) * 8, b_lk = ((lane >> 3) & 1) * 8;
+  for (int kb = 0; kb < nk; ++kb) {
+    const int st = kb % EF_STAGES;
+    asm volatile("cp.async.wait_group %0;" ::"n"(EF_STAGES - 2) : "memory");   // block kb has landed
+    __syncthreads();                                                           // and the stage of block kb - 1 is free
+    if (kb + EF_STAGES - 1 < nk) load_stage((kb + EF_STAGES - 1) % EF_STAGES, (kb + EF_STAGES - 1) * EF_BK);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll
+    for (int kk = 0; kk < EF_BK; kk += 16) {
+      uint32_t a[4], b0, b1, b2, b3;
+      ex_ldmatrix_x4(As + (st * EF_BM + a_lr) * EF_LD + kk + a_lk, a[0], a[1], a[2], a[3]);
+      ex_ldmatrix_x4(Bs + (st * EF_BN + wn + b_lr) * EF_LD + kk + b_lk, b0, b1, b2, b3);
+      const uint32_t lo[2] = {b0, b1}, hi[2] = {b2, b3};
+      ex_mma_16816(acc[0], a, lo);
+      ex_mma_16816(acc[1], a, hi);
+    }
+  }
+  TY* y = (TY*)p.y;
+#pragma unroll
+  for (int nb = 0; nb < 2; ++nb)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int row = r0 + (lane >> 2) + 8 * half;
+      if (row >= r1) continue;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const int n = n0 + wn + nb * 8 + 2 * (lane & 3) + j;
+        if (n < p.N) y[(size_t)row * p.ldy + n] = from_f32<TY>(post_op(p.post, 0.f, acc[nb][2 * half + j]));
+      }
+    }
+}
+
 // ---- combine ---------------------------------------------------------------------------------------------------
 // weights: null means `weight` for every pair.  gate (with x, the rows the products read): the always-used expert's output
 // counts times sigmoid(gate . x[t]).
@@ -488,19 +565,21 @@ LB_EXPORT int lb_route_topk(int* ids, float* weights, const float* logits, long 
   return 0;
 }
 
-// The row tiles of the experts' products have this many places.
-LB_EXPORT int lb_expert_tile_rows() { return lb::EX_BM; }
+// The row tiles of the experts' products have this many places; those of steps with a few pairs an expert `few` of them.
+LB_EXPORT int lb_expert_tile_rows(int few) { return few ? lb::EF_BM : lb::EX_BM; }
 
 // ids [pairs] -> offsets [experts + 1], pair_at [pairs], place_of [pairs], meta [4 + 3 * (pairs / tile_rows + experts)]
 // (tokens != null: ids is the table [vocab, top] and pairs = tokens * top; its entries lie in 0 .. experts - 1)
-LB_EXPORT int lb_expert_dispatch(const int* ids, const int* tokens, int top, int pairs, int experts, int* offsets, int* pair_at,
+// tile_rows: lb_expert_tile_rows of the product that will walk the tiles
+LB_EXPORT int lb_expert_dispatch(const int* ids, const int* tokens, int top, int pairs, int experts, int tile_rows, int* offsets, int* pair_at,
                                  int* place_of, int* meta, cudaStream_t stream) {
+  LB_CHECK_ARG(tile_rows == lb::EX_BM || tile_rows == lb::EF_BM, "expert_dispatch: row tiles of %d places", tile_rows);
   LB_CHECK_ARG(tokens == nullptr || (top > 0 && pairs % top == 0), "expert_dispatch: %d pairs are not %d choices a token", pairs, top);
   LB_CHECK_ARG(ids && offsets && pair_at && place_of && meta, "expert_dispatch: null argument");
   LB_CHECK_ARG(pairs >= 0 && experts > 0 && experts <= 4096, "expert_dispatch: bad sizes pairs=%d experts=%d", pairs, experts);
   static_assert(lb::EX_BM == lb::EM_BM, "both products walk the same row tiles");
   const size_t smem = (size_t)(3 * experts + 2) * sizeof(int);
-  lb::launch(lb::expert_dispatch_kernel, dim3(1), dim3(1024), smem, stream, ids, tokens, top, pairs, experts, (int)lb::EX_BM, offsets, pair_at, place_of, meta);
+  lb::launch(lb::expert_dispatch_kernel, dim3(1), dim3(1024), smem, stream, ids, tokens, top, pairs, experts, tile_rows, offsets, pair_at, place_of, meta);
   LB_CHECK_LAUNCH("expert_dispatch");
   return 0;
 }
@@ -532,7 +611,7 @@ LB_EXPORT int lb_expert_gather_rows(void* xs, const void* x, const int* pair_at,
 // fast: 1 allows the tensor-core kernel (bfloat16 x and W, K a multiple of 8, 16-byte aligned rows).
 LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* meta,
                              const int* pair_at, int max_tiles, int N, int K, long long ldx, long long ldy, int top, int gather,
-                             int gated, int act, float limit, int fast, int interleaved, int post, cudaStream_t stream) {
+                             int gated, int act, float limit, int fast, int interleaved, int post, int few, cudaStream_t stream) {
   LB_CHECK_ARG(lb::valid_post(post, 0.f) && !(post && gated), "expert_gemm: element operation %d", post);
   LB_CHECK_ARG(!interleaved || (gated && N % 128 == 0), "expert_gemm: interleaved gate and up rows come in blocks of 64");
   LB_CHECK_ARG(lb::valid_dtype(y_dtype) && lb::valid_dtype(x_dtype) && lb::valid_dtype(w_dtype), "expert_gemm: bad dtype");
@@ -546,7 +625,17 @@ LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, c
   p.gather = gather; p.gated = gated; p.act = act; p.limit = limit; p.interleaved = interleaved; p.post = post;
   const int ncols = gated ? N / 2 : N;
   const bool mma = fast && x_dtype == LB_BF16 && w_dtype == LB_BF16 && K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0;
-  if (mma) {
+  LB_CHECK_ARG(!few || (mma && !gated), "expert_gemm: tiles of a few places are for ungated bfloat16 products on the tensor cores");
+  if (few) {
+    static bool few_set = false;
+    if (!few_set) {
+      cudaFuncSetAttribute(lb::expert_gemm_few_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::EF_SMEM);
+      cudaFuncSetAttribute(lb::expert_gemm_few_kernel<lb::bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::EF_SMEM);
+      few_set = true;
+    }
+    dim3 grid((N + lb::EF_BN - 1) / lb::EF_BN, max_tiles);
+    LB_DISPATCH_DTYPE(y_dtype, TY, { lb::launch(lb::expert_gemm_few_kernel<TY>, grid, dim3(128), lb::EF_SMEM, stream, p); })
+  } else if (mma) {
     static bool attr_set = false;
     if (!attr_set) {       // the stages need more shared memory than a launch gets unasked
       cudaFuncSetAttribute(lb::expert_gemm_mma_kernel<float, true, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::expert_mma_smem<true, 128>());

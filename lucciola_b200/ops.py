@@ -45,9 +45,9 @@ _SIGNATURES = {
                          c_int, c_longlong, c_void_p],
     "lb_head_gate": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_longlong, c_float, c_int, c_int, c_int, c_void_p],
     "lb_route_topk": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
-    "lb_expert_dispatch": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
+    "lb_expert_dispatch": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "lb_expert_gemm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong,
-                       c_longlong, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_void_p],
+                       c_longlong, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p],
     "lb_expert_dispatch_padded": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "lb_expert_gather_rows": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lb_gemm_tcgen05_grouped": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_int, c_float,
@@ -923,15 +923,17 @@ def route_topk(ids: torch.Tensor, weights: torch.Tensor, logits: torch.Tensor, c
           T, E, ids.shape[1], groups, keep, scale, stream)
 
 
-def expert_tile_rows() -> int:
+def expert_tile_rows(few: bool = False) -> int:
+    """Places of a row tile of the experts' products; `few`: of those for steps with a few pairs an expert."""
     lib = library()
+    lib.lb_expert_tile_rows.argtypes = [c_int]
     lib.lb_expert_tile_rows.restype = c_int
-    return int(lib.lb_expert_tile_rows())
+    return int(lib.lb_expert_tile_rows(1 if few else 0))
 
 
-def expert_max_tiles(pairs: int, experts: int) -> int:
+def expert_max_tiles(pairs: int, experts: int, few: bool = False) -> int:
     """The most row tiles the experts' products can have for this many (token, choice) pairs."""
-    return -(-pairs // expert_tile_rows()) + experts
+    return -(-pairs // expert_tile_rows(few)) + experts
 
 
 def _dispatch_pairs(ids: torch.Tensor, tokens: torch.Tensor | None) -> tuple[int, int]:
@@ -942,26 +944,28 @@ def _dispatch_pairs(ids: torch.Tensor, tokens: torch.Tensor | None) -> tuple[int
 
 
 def expert_dispatch(ids: torch.Tensor, experts: int, offsets: torch.Tensor, pair_at: torch.Tensor, place_of: torch.Tensor,
-                    meta: torch.Tensor, stream: int, tokens: torch.Tensor | None = None) -> None:
+                    meta: torch.Tensor, stream: int, tokens: torch.Tensor | None = None, few: bool = False) -> None:
     """Sort the (token, choice) pairs by expert, on the device: offsets [experts + 1], pair_at [pairs] (the pair at each
     place), place_of [pairs], meta [4 + 3 * expert_max_tiles] (the row tiles of the products).  ids: the experts of the pairs, [T, top], or, with the step's
-    `tokens` [T], a table [vocab, top] whose row of a token's id holds the token's experts (entries in 0 .. experts - 1)."""
+    `tokens` [T], a table [vocab, top] whose row of a token's id holds the token's experts (entries in 0 .. experts - 1).
+    `few`: row tiles for expert_gemm(few=True)."""
     for t, what in ((ids, "expert ids"), (offsets, "offsets"), (pair_at, "pair list"), (place_of, "places"), (meta, "tile list")):
         _check(t, what, torch.int32)
     pairs, top = _dispatch_pairs(ids, tokens)
-    if offsets.numel() < experts + 1 or pair_at.numel() < pairs or place_of.numel() < pairs or meta.numel() < 4 + 3 * expert_max_tiles(pairs, experts):
+    if offsets.numel() < experts + 1 or pair_at.numel() < pairs or place_of.numel() < pairs or meta.numel() < 4 + 3 * expert_max_tiles(pairs, experts, few):
         raise KernelError("expert_dispatch: an output is too small")
-    _call("lb_expert_dispatch", ids.data_ptr(), _ptr(tokens), top, pairs, experts, offsets.data_ptr(), pair_at.data_ptr(), place_of.data_ptr(),
+    _call("lb_expert_dispatch", ids.data_ptr(), _ptr(tokens), top, pairs, experts, expert_tile_rows(few), offsets.data_ptr(), pair_at.data_ptr(), place_of.data_ptr(),
           meta.data_ptr(), stream)
 
 
 def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, pair_at: torch.Tensor, top: int,
                 gather: bool, stream: int, act: str | None = None, limit: float = 0.0, fast: bool = True,
-                interleaved: bool = False, post: str | None = None) -> None:
+                interleaved: bool = False, post: str | None = None, few: bool = False) -> None:
     """y[place] = x[row(place)] . w[e]^T for the places of every expert e (see expert_dispatch); w [experts, N, K].
     `gather`: row(place) is the pair's token, else the place.  With `act`, w[e] is N/2 gate rows then N/2 up rows (or,
     `interleaved`, blocks of 64 gate rows and their 64 up rows in turn, see interleave_gate_up) and y[place] =
-    act(gate) * up with N/2 columns.  `post` (without act): an element operation on the sums, see POST_OPS."""
+    act(gate) * up with N/2 columns.  `post` (without act): an element operation on the sums, see POST_OPS.
+    `few` (without act, bfloat16): row tiles of few places, see expert_dispatch; the weights then stream through a kernel of their own."""
     _check(y, "expert output"); _check(x, "expert input"); _check(w, "expert weights")
     E, N, K = w.shape
     pairs = pair_at.numel()
@@ -969,9 +973,9 @@ def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.T
     if x.shape[1] != K or y.shape[1] != cols or y.shape[0] != pairs:
         raise KernelError(f"expert_gemm shapes do not fit: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     _call("lb_expert_gemm", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), dtype_code(x.dtype), w.data_ptr(), dtype_code(w.dtype),
-          meta.data_ptr(), pair_at.data_ptr(), expert_max_tiles(pairs, E), N, K, K, cols, top, 1 if gather else 0,
+          meta.data_ptr(), pair_at.data_ptr(), expert_max_tiles(pairs, E, few), N, K, K, cols, top, 1 if gather else 0,
           1 if act is not None else 0, GATE_ACTS[act] if act is not None else 0, limit, 1 if fast else 0, 1 if interleaved else 0,
-          POST_OPS[post], stream)
+          POST_OPS[post], 1 if few else 0, stream)
 
 
 GROUP_TILE = 128          # token tile of the grouped tensor-memory product

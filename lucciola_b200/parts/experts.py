@@ -39,6 +39,9 @@ from .linear import Linear
 # From this many pairs of token and choice an expert (on average) the padded runs of the tensor-memory product cost
 # less than they gain: the padding is 64 places an expert on average, 127 at most, and the product several times faster.
 GROUPED_FROM = 96
+# Up to this many pairs an expert (on average) an ungated step is a stream of the experts' weights and takes the kernel made for
+# it, whose row tiles have 16 places (an expert with more reads its weights once a tile).
+FEW_UP_TO = 8
 
 
 @dataclass
@@ -48,6 +51,7 @@ class Dispatch:
     place_of: torch.Tensor
     meta: Optional[torch.Tensor] = None             # the row tiles of the runs; None: runs padded to whole tiles, then
     tile_group: Optional[torch.Tensor] = None       # the expert of each tile
+    few: bool = False                               # row tiles of few places
 
 
 class ExpertBank(FeedForward):
@@ -102,9 +106,10 @@ class ExpertBank(FeedForward):
             ops.expert_dispatch_padded(ids, E, pair_at, place_of, tile_group, rt.stream, tokens=tokens)
             return Dispatch(pair_at, place_of, tile_group=tile_group)
         offsets, pair_at = rt.empty((E + 1,), torch.int32), rt.empty((pairs,), torch.int32)
-        meta = rt.empty((4 + 3 * ops.expert_max_tiles(pairs, E),), torch.int32)
-        ops.expert_dispatch(ids, E, offsets, pair_at, place_of, meta, rt.stream, tokens=tokens)
-        return Dispatch(pair_at, place_of, meta=meta)
+        few = self.grouped_ok and not self.gated and pairs <= FEW_UP_TO * E
+        meta = rt.empty((4 + 3 * ops.expert_max_tiles(pairs, E, few),), torch.int32)
+        ops.expert_dispatch(ids, E, offsets, pair_at, place_of, meta, rt.stream, tokens=tokens, few=few)
+        return Dispatch(pair_at, place_of, meta=meta, few=few)
 
     def products(self, h: torch.Tensor, d: Dispatch) -> torch.Tensor:
         """The experts' outputs at their places, float32 [places, width]."""
@@ -119,8 +124,8 @@ class ExpertBank(FeedForward):
             ops.gemm_tcgen05_grouped(y, inner, self.down, d.tile_group, rt.stream)
             return y
         ops.expert_gemm(inner, h, self.gate_up, d.meta, d.pair_at, self.top, True, rt.stream, fast=rt.fast_kernels,
-                        interleaved=self.interleaved, **how)
-        ops.expert_gemm(y, inner, self.down, d.meta, d.pair_at, self.top, False, rt.stream, fast=rt.fast_kernels)
+                        interleaved=self.interleaved, few=d.few, **how)
+        ops.expert_gemm(y, inner, self.down, d.meta, d.pair_at, self.top, False, rt.stream, fast=rt.fast_kernels, few=d.few)
         return y
 
 
