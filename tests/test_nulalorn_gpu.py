@@ -200,7 +200,7 @@ def test_element_operations_in_the_products(post, c, M, N, K):
 
 @pytest.mark.parametrize("dtype", TYPES)
 @pytest.mark.parametrize("experts,top,width,ff,shared,lens", [(5, 2, 74, 28, 36, [3, 1, 9]), (1, 1, 40, 32, None, [1]), (16, 4, 256, 64, 64, [1] * 8), (16, 4, 200, 72, None, [5]), (4, 1, 128, 520, 24, [30]), (40, 2, 64, 16, None, [90, 3]),
-                                                              (2, 2, 256, 64, 128, [130, 70]), (6, 1, 128, 136, 24, [700]), (3, 3, 64, 12, 20, [300, 5])])
+                                                              (2, 2, 256, 64, 128, [130, 70]), (6, 1, 128, 152, 24, [700]), (3, 3, 64, 12, 20, [300, 5])])
 def test_experts_named_by_a_table(dtype, experts, top, width, ff, shared, lens):
     """Short runs of tokens and runs long enough for the tensor-memory product (bfloat16), summed in the norm's kernel and
     alone; an expert that nobody names; a second call in one step uses the first one's sorting."""
