@@ -1,7 +1,7 @@
 // Plain paged attention: one warp per (query token, query head), keys visited
 // in their order in the sequence, everything in 32-bit.  It serves the 32-bit
 // path of the engine and is the kernel beside which the fast bfloat16 kernels
-// are tested.  It takes any head size up to 512, any head counts and group
+// are tested.  It takes any head size up to 3072 (values up to 1024), any head counts and group
 // sizes, any page size, whole prompts, portions and single decoded tokens alike.
 //
 // Formulas as in lucciola: kv head = q head / (nq / nkv)
@@ -13,7 +13,8 @@
 // holds cannot reach a sum.
 //
 // Two more things lucciola does not have.  Values may have another size than keys (v_dim; the value pool is
-// then [page][kv_head][slot][v_dim]).  And a linear distance bias: with `slopes` (one 32-bit number a query
+// then [page][kv_head][slot][v_dim], or its rows are `v_stride` apart: values that are the first v_dim entries of
+// longer rows, as with a latent whose keys carry a rotated part behind it).  And a linear distance bias: with `slopes` (one 32-bit number a query
 // head) the score of key j for the query at position i is (q . k) * scale - slopes[h] * (i - j).
 //
 // Three more options.  A capped score: s <- softcap * tanh(s / softcap).  A sink: with `sinks` (one 32-bit number a
@@ -34,6 +35,7 @@ struct PlainAttnParams {
   int num_q_heads, num_kv_heads, head_dim, page_size, max_pages, window;
   float scale;
   int v_dim;               // size of a value head
+  int v_stride;            // entries between the value pool's rows
   const float* slopes;     // optional [num_q_heads]: distance bias
   float softcap;           // 0: scores are not capped
   const float* sinks;      // optional [num_q_heads]
@@ -102,7 +104,7 @@ __global__ void plain_attention_kernel(PlainAttnParams p) {
         const float pv = __shfl_sync(0xffffffffu, pj, jj);
         const long long voff = __shfl_sync(0xffffffffu, off, jj);
         if (voff < 0) continue;  // uniform over the warp
-        const T* v = vc + voff * dv;
+        const T* v = vc + voff * p.v_stride;
 #pragma unroll
         for (int i = 0; i < DPL; ++i) {
           const int dim = lane + 32 * i;
@@ -146,7 +148,8 @@ int launch_plain(const PlainAttnParams& p, int num_tokens, cudaStream_t stream) 
   else if (dpl <= 2) launch(plain_attention_kernel<T, 2>, grid, dim3(warps * 32), smem, stream, p);
   else if (dpl <= 4) launch(plain_attention_kernel<T, 4>, grid, dim3(warps * 32), smem, stream, p);
   else if (dpl <= 8) launch(plain_attention_kernel<T, 8>, grid, dim3(warps * 32), smem, stream, p);
-  else launch(plain_attention_kernel<T, 16>, grid, dim3(warps * 32), smem, stream, p);
+  else if (dpl <= 16) launch(plain_attention_kernel<T, 16>, grid, dim3(warps * 32), smem, stream, p);
+  else launch(plain_attention_kernel<T, 32>, grid, dim3(warps * 32), smem, stream, p);
   return 0;
 }
 
@@ -158,15 +161,16 @@ LB_EXPORT int lb_attention_plain(int dtype, const void* q, void* out, const void
                                  int num_kv_heads, int head_dim, int page_size, int max_pages,
                                  int window, float scale, int v_dim, const float* slopes, float softcap,
                                  const float* sinks, int pool, const void* pool_k, const void* pool_v, const int* pool_table,
-                                 int pool_max_pages, int chunk, cudaStream_t stream) {
+                                 int pool_max_pages, int chunk, int v_stride, cudaStream_t stream) {
   LB_CHECK_ARG(chunk >= 0 && (chunk == 0 || pool == 0), "attention_plain: chunks of %d keys (and no pooled blocks with them)", chunk);
   LB_CHECK_ARG(pool == 0 || (pool > 0 && window > 0 && pool_k && pool_v && pool_table && pool_max_pages > 0),
                "attention_plain: pooled blocks need a window, the pooled cache and its block table");
   LB_CHECK_ARG(softcap >= 0.f, "attention_plain: a cap of %f", (double)softcap);
   if (v_dim <= 0) v_dim = head_dim;
-  LB_CHECK_ARG(v_dim <= 512, "attention_plain: value size %d not in 1..512", v_dim);
+  if (v_stride <= 0) v_stride = v_dim;
+  LB_CHECK_ARG(v_dim <= 1024 && v_stride >= v_dim, "attention_plain: value size %d not in 1..1024, or rows of %d", v_dim, v_stride);
   LB_CHECK_ARG(lb::valid_dtype(dtype), "attention_plain: bad dtype %d", dtype);
-  LB_CHECK_ARG(head_dim > 0 && head_dim <= 512, "attention_plain: head_dim %d not in 1..512", head_dim);
+  LB_CHECK_ARG(head_dim > 0 && head_dim <= 3072, "attention_plain: head_dim %d not in 1..3072", head_dim);
   LB_CHECK_ARG(num_q_heads > 0 && num_kv_heads > 0 && num_q_heads % num_kv_heads == 0,
                "attention_plain: %d query heads are not a multiple of %d kv heads", num_q_heads,
                num_kv_heads);
@@ -179,7 +183,7 @@ LB_EXPORT int lb_attention_plain(int dtype, const void* q, void* out, const void
   p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.head_dim = head_dim;
   p.page_size = page_size; p.max_pages = max_pages; p.window = window; p.scale = scale; p.v_dim = v_dim; p.slopes = slopes;
   p.softcap = softcap; p.sinks = sinks; p.pool = pool; p.pool_k = pool_k; p.pool_v = pool_v; p.pool_table = pool_table;
-  p.pool_max_pages = pool_max_pages; p.chunk = chunk;
+  p.pool_max_pages = pool_max_pages; p.chunk = chunk; p.v_stride = v_stride;
   LB_DISPATCH_DTYPE(dtype, T, { lb::launch_plain<T>(p, num_tokens, stream); })
   LB_CHECK_LAUNCH("attention_plain");
   return 0;

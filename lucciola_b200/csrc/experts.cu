@@ -35,7 +35,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 
 __global__ void route_topk_kernel(int* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
                                   long long ld, const float* __restrict__ correction, int num_tokens, int experts, int top,
-                                  int groups, int keep, float scale) {
+                                  int groups, int keep, float scale, int softmax) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -47,7 +47,8 @@ __global__ void route_topk_kernel(int* __restrict__ ids, float* __restrict__ wei
   float* gw = c + experts;                          // what a group is worth; then the sum of the chosen scores
   const int size = experts / groups;
   for (int e = lane; e < experts; e += 32) {
-    const float v = 1.f / (1.f + expf(-logits[(size_t)t * ld + e]));
+    const float z = logits[(size_t)t * ld + e];
+    const float v = softmax ? z : 1.f / (1.f + expf(-z));
     s[e] = v;
     c[e] = v + (correction ? correction[e] : 0.f);
   }
@@ -77,7 +78,7 @@ __global__ void route_topk_kernel(int* __restrict__ ids, float* __restrict__ wei
       if (gw[e / size] != INFINITY) c[e] = -INFINITY;
     __syncwarp();
   }
-  float sum = 0.f;                                    // the same on every lane
+  float sum = 0.f, best = 0.f;                        // the same on every lane
   for (int r = 0; r < top; ++r) {
     float bv = -INFINITY; int bi = 0x7fffffff;
     for (int e = lane; e < experts; e += 32) {
@@ -86,12 +87,20 @@ __global__ void route_topk_kernel(int* __restrict__ ids, float* __restrict__ wei
     }
     warp_argmax(bv, bi);
     if (bi >= experts) bi = 0;                        // nothing left to choose from: cannot happen with top <= keep * size
-    sum += s[bi];
+    if (softmax) {                                    // the first chosen is the largest: the reference of the exponentials
+      if (r == 0) best = s[bi];
+      sum += expf(s[bi] - best);
+    } else {
+      sum += s[bi];
+    }
     if (lane == 0) { ids[(size_t)t * top + r] = bi; c[bi] = NAN; }      // NaN marks a chosen expert (-inf is a legal score)
     __syncwarp();
   }
   const float f = scale / (sum + 1e-20f);
-  for (int r = lane; r < top; r += 32) weights[(size_t)t * top + r] = s[ids[(size_t)t * top + r]] * f;
+  for (int r = lane; r < top; r += 32) {
+    const float v = s[ids[(size_t)t * top + r]];
+    weights[(size_t)t * top + r] = (softmax ? expf(v - best) : v) * f;
+  }
 }
 
 // ---- dispatch --------------------------------------------------------------------------------------------------
@@ -551,7 +560,8 @@ __global__ void expert_combine_kernel(TO* __restrict__ out, const float* __restr
 
 // ids [T, top] int32, weights [T, top] float32 from logits [T, ld] float32 and correction [experts] float32 (may be null)
 LB_EXPORT int lb_route_topk(int* ids, float* weights, const float* logits, long long ld, const float* correction,
-                            int num_tokens, int experts, int top, int groups, int keep, float scale, cudaStream_t stream) {
+                            int num_tokens, int experts, int top, int groups, int keep, float scale, int softmax, cudaStream_t stream) {
+  LB_CHECK_ARG(!softmax || correction == nullptr, "route_topk: no correction of the choice with softmax weights");
   LB_CHECK_ARG(ids && weights && logits, "route_topk: null argument");
   LB_CHECK_ARG(num_tokens >= 0 && experts > 0 && experts <= 4096 && top > 0 && top <= experts && groups > 0 && experts % groups == 0 &&
                keep > 0 && keep <= groups && top <= keep * (experts / groups) && ld >= experts,
@@ -560,7 +570,7 @@ LB_EXPORT int lb_route_topk(int* ids, float* weights, const float* logits, long 
   const int warps = experts > 1024 ? 1 : 4;
   const size_t smem = (size_t)warps * 3 * experts * sizeof(float);
   lb::launch(lb::route_topk_kernel, dim3((num_tokens + warps - 1) / warps), dim3(warps * 32), smem, stream, ids, weights, logits, ld,
-             correction, num_tokens, experts, top, groups, keep, scale);
+             correction, num_tokens, experts, top, groups, keep, scale, softmax);
   LB_CHECK_LAUNCH("route_topk");
   return 0;
 }

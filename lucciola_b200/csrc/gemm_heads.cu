@@ -1,6 +1,6 @@
 // One product a head on the tensor cores: y[m, b, :] = x[m, b, :] . w[b]^T for b < batches (the heads of a mixer
 // whose heads each have a matrix of their own), bfloat16 operands, 32-bit sums, optionally times
-// sigmoid(gate[m, b * N + n]) (32-bit gate) before the single rounding.  Tiles of 64 x 64 outputs a CTA of four
+// sigmoid(gate[m, b * N + n]) (32-bit gate; or one gate a batch, gate[m, b]) before the single rounding.  Tiles of 64 x 64 outputs a CTA of four
 // warps (mma.sync m16n8k16: these products are small and many, K is a head's size or a latent's), operands
 // staged through shared memory in blocks of 64 along K.  K must be a multiple of 8 and the operands 16-byte
 // aligned; other shapes go to the plain kernel.
@@ -19,7 +19,7 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a
 __global__ void __launch_bounds__(128)
 gemm_heads_mma_kernel(bf16* __restrict__ y, const bf16* __restrict__ x, const bf16* __restrict__ w, int M, int N, int K,
                       long long ldx, long long ldy, long long bx, long long bw, long long by,
-                      const float* __restrict__ gate, long long ldg) {
+                      const float* __restrict__ gate, long long ldg, int gate_one) {
   __shared__ __align__(16) bf16 As[GH_BM][GH_LD];
   __shared__ __align__(16) bf16 Bs[GH_BN][GH_LD];
   pdl_trigger();
@@ -66,7 +66,7 @@ gemm_heads_mma_kernel(bf16* __restrict__ y, const bf16* __restrict__ x, const bf
     }
     __syncthreads();
   }
-  if (gate) gate += (size_t)b * N;
+  if (gate) gate += gate_one ? (size_t)b : (size_t)b * N;
 #pragma unroll
   for (int nb = 0; nb < 8; ++nb) {
 #pragma unroll
@@ -78,7 +78,7 @@ gemm_heads_mma_kernel(bf16* __restrict__ y, const bf16* __restrict__ x, const bf
         const int n = n0 + nb * 8 + 2 * t4 + j;
         if (n >= N) continue;
         float v = acc[nb][2 * half + j];
-        if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)m * ldg + n]));
+        if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)m * ldg + (gate_one ? 0 : n)]));
         y[(size_t)m * ldy + n] = __float2bfloat16_rn(v);
       }
     }
@@ -94,16 +94,16 @@ LB_EXPORT int lb_gemm_heads_mma_ok(const void* y, const void* x, const void* w, 
 
 LB_EXPORT int lb_gemm_heads_mma(void* y, const void* x, const void* w, int batches, int M, int N, int K, long long ldx,
                                 long long ldy, long long bx, long long bw, long long by, const float* gate, long long ldg,
-                                cudaStream_t stream) {
+                                int gate_one, cudaStream_t stream) {
   LB_CHECK_ARG(M >= 0 && N > 0 && K > 0 && batches > 0 && batches <= 65535 && ldx >= K && ldy >= N,
                "gemm_heads_mma: bad sizes batches=%d M=%d N=%d K=%d", batches, M, N, K);
   LB_CHECK_ARG(lb_gemm_heads_mma_ok(y, x, w, K, ldx, bx, bw), "gemm_heads_mma: K, strides and addresses must be multiples of 8 values (16 bytes)");
-  LB_CHECK_ARG(gate == nullptr || ldg >= (long long)batches * N, "gemm_heads_mma: the gate's rows are shorter than batches * N");
+  LB_CHECK_ARG(gate == nullptr || ldg >= (long long)batches * (gate_one ? 1 : N), "gemm_heads_mma: the gate's rows are too short");
   LB_CHECK_ARG((M + lb::GH_BM - 1) / lb::GH_BM <= 65535, "gemm_heads_mma: too many rows (%d)", M);
   if (M == 0) return 0;
   dim3 grid((N + lb::GH_BN - 1) / lb::GH_BN, (M + lb::GH_BM - 1) / lb::GH_BM, batches);
   lb::launch(lb::gemm_heads_mma_kernel, grid, dim3(128), 0, stream, (lb::bf16*)y, (const lb::bf16*)x, (const lb::bf16*)w, M, N, K,
-             ldx, ldy, bx, bw, by, gate, ldg);
+             ldx, ldy, bx, bw, by, gate, ldg, gate_one);
   LB_CHECK_LAUNCH("gemm_heads_mma");
   return 0;
 }

@@ -15,6 +15,7 @@
 //
 // Two more forms lucciola does not have.  `pairs`: the pairs are neighbours, (2i, 2i + 1), instead of (i, i + rot/2).
 // `unit`: after the rotation every q and k head is divided by its root mean square (sqrt(mean(x^2) + eps), no weight).
+// And a query temperature: behind all that the queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).
 #include "common.cuh"
 
 #include <type_traits>
@@ -35,7 +36,13 @@ struct RopeKvParams {
   float rot_scale;                           // sines and cosines are multiplied by this (1: a pure rotation)
   int pairs;                                 // 1: neighbours (2i, 2i + 1) are a pair, not (i, i + rot/2)
   int unit;                                  // 1: divided by the root mean square behind the rotation, without a weight
+  float temp_coef; int temp_every;           // temp_every > 0: queries are multiplied by their position's temperature
 };
+
+// 1 + coef * ln(floor((p + 1) / every) + 1), or 1 without a temperature.
+__device__ __forceinline__ float query_temperature(const RopeKvParams& p, int pos) {
+  return p.temp_every > 0 ? 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1)) : 1.f;
+}
 
 // TI: the type of q_in, k_in, v_in (a product's output, which may be 32-bit where the heads are stored in bfloat16)
 template <typename T, typename TI>
@@ -48,6 +55,7 @@ __global__ void rope_kv_kernel(RopeKvParams p) {
   const int d = p.head_dim, dv = p.v_dim, half = p.rot_dim >> 1;
   float* buf = smem + (size_t)warp * d;
   const int pos = p.positions[t];
+  const float temp = query_temperature(p, pos);
   const int total_heads = p.num_q_heads + 2 * p.num_kv_heads;
 
   // One head per warp: the grid's second dimension covers the heads.
@@ -94,7 +102,7 @@ __global__ void rope_kv_kernel(RopeKvParams p) {
       for (int i = lane; i < d; i += 32) buf[i] = buf[i] * inv * w[i];
       __syncwarp();
     }
-    if (p.pairs || p.unit) {
+    if (p.pairs || p.unit || p.temp_every > 0) {
       // rotated in place in shared memory, then divided, then stored
       if (p.inv_freq) {
         for (int i = lane; i < half; i += 32) {
@@ -114,6 +122,7 @@ __global__ void rope_kv_kernel(RopeKvParams p) {
         for (int i = lane; i < d; i += 32) s2 += buf[i] * buf[i];
         f = rsqrtf(warp_sum(s2) / (float)d + p.eps);
       }
+      if (kind == 0) f *= temp;
       for (int i = lane; i < d; i += 32) dst[i] = from_f32<T>(buf[i] * f);
     } else if (p.inv_freq) {
       for (int i = lane; i < half; i += 32) {
@@ -250,6 +259,7 @@ __global__ void rope_pairs_kernel(RopeKvParams p) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   const int d = p.head_dim, dv = p.v_dim;
   const int pos = p.positions[t];
+  const float temp = query_temperature(p, pos);
   const int total_heads = p.num_q_heads + 2 * p.num_kv_heads;
   float2 cs[NV], sn[NV];
 #pragma unroll
@@ -331,8 +341,8 @@ __global__ void rope_pairs_kernel(RopeKvParams p) {
                                 a.z * cs[n].y - a.w * sn[n].y, a.z * sn[n].y + a.w * cs[n].y);
           ss += x[u][n].x * x[u][n].x + x[u][n].y * x[u][n].y + x[u][n].z * x[u][n].z + x[u][n].w * x[u][n].w;
         }
-        if (p.unit) {
-          const float f = rsqrtf(warp_sum(ss) / (float)d + p.eps);
+        if (p.unit || (kind == 0 && p.temp_every > 0)) {
+          const float f = (p.unit ? rsqrtf(warp_sum(ss) / (float)d + p.eps) : 1.f) * (kind == 0 ? temp : 1.f);
 #pragma unroll
           for (int n = 0; n < NV; ++n) { x[u][n].x *= f; x[u][n].y *= f; x[u][n].z *= f; x[u][n].w *= f; }
         }
@@ -412,7 +422,7 @@ LB_EXPORT int lb_rope_kv(int dtype, const void* q_in, const void* k_in, const vo
                          const float* q_norm_w, const float* k_norm_w, const float* inv_freq,
                          int num_tokens, int num_q_heads, int num_kv_heads, int head_dim,
                          int rot_dim, int page_size, int max_pages, float eps, int in_dtype, int v_dim,
-                         float rot_scale, int pairs, int unit, cudaStream_t stream) {
+                         float rot_scale, int pairs, int unit, float temp_coef, int temp_every, cudaStream_t stream) {
   if (v_dim <= 0) v_dim = head_dim;
   LB_CHECK_ARG(lb::valid_dtype(in_dtype) && v_dim <= 1024, "rope_kv: bad input type or value size");
   LB_CHECK_ARG(lb::valid_dtype(dtype), "rope_kv: bad dtype %d", dtype);
@@ -431,10 +441,12 @@ LB_EXPORT int lb_rope_kv(int dtype, const void* q_in, const void* k_in, const vo
   p.q_norm_w = q_norm_w; p.k_norm_w = k_norm_w; p.inv_freq = rot_dim > 0 ? inv_freq : nullptr;
   p.num_q_heads = num_q_heads; p.num_kv_heads = num_kv_heads; p.head_dim = head_dim;
   p.rot_dim = rot_dim; p.page_size = page_size; p.max_pages = max_pages; p.eps = eps; p.v_dim = v_dim;
-  p.rot_scale = rot_scale; p.pairs = pairs; p.unit = unit;
+  p.rot_scale = rot_scale; p.pairs = pairs; p.unit = unit; p.temp_coef = temp_coef; p.temp_every = temp_every;
+  LB_CHECK_ARG(temp_every >= 0, "rope_kv: a temperature that grows every %d positions", temp_every);
   LB_CHECK_ARG(!unit || (q_norm_w == nullptr && k_norm_w == nullptr), "rope_kv: heads are normed in front of the rotation or behind it, not both");
   const int warps = 4;
-  if (pairs && head_dim % 4 == 0 && v_dim % 4 == 0 && head_dim <= 256 && v_dim <= 256) {
+  // (without a rotation how entries pair does not matter: that kernel then serves unit heads of either kind)
+  if ((pairs || (unit && p.inv_freq == nullptr)) && head_dim % 4 == 0 && v_dim % 4 == 0 && head_dim <= 256 && v_dim <= 256) {
     const int in_el = in_dtype == LB_F32 ? 4 : 2, el = dtype == LB_F32 ? 4 : 2;
     auto in_ok = [&](const void* ptr, long long stride) { return (uintptr_t)ptr % (4 * in_el) == 0 && stride % 4 == 0; };
     auto out_ok = [&](const void* ptr) { return (uintptr_t)ptr % (4 * el) == 0; };
@@ -461,7 +473,7 @@ LB_EXPORT int lb_rope_kv(int dtype, const void* q_in, const void* k_in, const vo
   const int vec = head_dim / 32;
   const size_t word = (size_t)vec * 2;
   auto aligned = [&](const void* ptr, long long stride) { return ptr == nullptr || ((uintptr_t)ptr % word == 0 && (stride * 2) % (long long)word == 0); };
-  const bool fast = !pairs && !unit && dtype == LB_BF16 && in_dtype == LB_BF16 && v_dim == head_dim && (head_dim == 64 || head_dim == 128 || head_dim == 256) &&
+  const bool fast = !pairs && !unit && temp_every == 0 && dtype == LB_BF16 && in_dtype == LB_BF16 && v_dim == head_dim && (head_dim == 64 || head_dim == 128 || head_dim == 256) &&
                     (p.inv_freq == nullptr || rot_dim == head_dim) && aligned(q_in, q_stride) && aligned(k_in, k_stride) &&
                     aligned(v_in, v_stride) && aligned(q_out, head_dim) && aligned(k_out, head_dim) && aligned(v_out, head_dim) &&
                     aligned(k_cache, head_dim) && aligned(v_cache, head_dim);

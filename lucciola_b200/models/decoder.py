@@ -15,7 +15,7 @@ from typing import Optional, Sequence
 import torch
 
 from .. import ops
-from ..parts.base import Block, KVPages, Norm, Part, Pending, Runtime, StateSlot, StepContext, StreamCopy
+from ..parts.base import Block, KVPages, Norm, Part, Pending, Runtime, StateSlot, StepContext, StreamCopy, StreamUpdate
 from ..parts.embedding import OutputHead, TokenEmbedding
 from ..parts.norm import pending_terms
 from ..parts.stream_entry import StreamEntry
@@ -79,6 +79,8 @@ class DecoderModel(Part):
 
     def _settle(self, residual: torch.Tensor, delta) -> None:
         """Add what a block left to the stream by a kernel of its own; nothing is left then."""
+        if isinstance(delta, StreamUpdate):
+            raise ops.KernelError("a block that keeps several residual streams stands in front of one that knows only one")
         if isinstance(delta, Pending):
             ops.stream_norm(residual, self.rt.stream, **pending_terms(delta))
         elif torch.is_tensor(delta) or isinstance(delta, tuple):
@@ -119,7 +121,7 @@ class DecoderModel(Part):
             block = self.blocks[c.block]
             if isinstance(delta, StreamCopy) and not block.takes_stream_copy:
                 delta = None                             # nothing is left to be added; this block makes its own input
-            if isinstance(delta, Pending) and not block.takes_pending:
+            if (isinstance(delta, Pending) and not block.takes_pending) or (isinstance(delta, StreamUpdate) and not block.takes_streams):
                 delta = self._settle(residual, delta)
             next_sink = (self.blocks[nxt.block].entry_sink(residual, step.num_tokens, nxt.write_cache)
                          if nxt is not None and not nxt.add_embedding and nxt.entry < 0 else None)
@@ -136,7 +138,7 @@ class DecoderModel(Part):
             return None
         if isinstance(delta, StreamCopy):
             delta = None
-        if isinstance(delta, Pending) and not self.final_norm.takes_pending:
+        if (isinstance(delta, Pending) and not self.final_norm.takes_pending) or (isinstance(delta, StreamUpdate) and not self.final_norm.takes_streams):
             delta = self._settle(residual, delta)
         h = self.final_norm.add_forward(residual, delta, self.rt.act_dtype, rows=logit_rows)
         return self.head.forward(h)

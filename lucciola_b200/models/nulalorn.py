@@ -4,7 +4,7 @@
     the layers in order, of which layers loop.start .. loop.stop - 1 run loop.times times in a row (same weights, a cache of
     its own for every pass; in front of pass t:  x <- W_in [x ; x0] + step[t]):                             (StreamEntry)
         x += n1b(mixer(n1(x)));   x += n2b(ffn(n2(x)))                  (SandwichNormBlock; a layer may have no ffn)
-        mixer: window attention with a capped score on rotated q and k of unit mean square       (CappedWindowAttention)
+        mixer: window attention with a capped score on rotated q and k of unit mean square       (UnitHeadAttention)
         ffn:   down(gelu(up h)), or such experts named by a table of the token ids, beside a shared one   (TableExperts)
     logits = cap(head . rmsnorm(x))
 
@@ -18,7 +18,7 @@ import torch
 
 from ..config.nulalorn_config import MOE, NeighbourRotarySpec, NulalornConfig
 from ..config.registry import register_architecture
-from ..parts.attention import CappedWindowAttention
+from ..parts.attention import UnitHeadAttention
 from ..parts.base import Runtime
 from ..parts.block import SandwichNormBlock
 from ..parts.embedding import OutputHead, TokenEmbedding
@@ -41,7 +41,7 @@ def build_nulalorn(cfg: NulalornConfig, rt: Runtime) -> DecoderModel:
     blocks = []
     for i, l in enumerate(cfg.layers):
         p, a, f = f"l{i}", l.attention, l.mlp
-        mixer = CappedWindowAttention(rt, f"{p}.mix", W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.softcap, _rotary(rt, a.dim, a.rot),
+        mixer = UnitHeadAttention(rt, f"{p}.mix", W, a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.softcap, _rotary(rt, a.dim, a.rot),
                                       a.window, eps, out_dtype=f32)
         ffn = None
         if f is not None and f.kind == MOE:

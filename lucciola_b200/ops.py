@@ -44,7 +44,11 @@ _SIGNATURES = {
     "lb_rmsnorm_gated": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_float, c_float, c_int, c_int,
                          c_int, c_longlong, c_void_p],
     "lb_head_gate": [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_longlong, c_float, c_int, c_int, c_int, c_void_p],
-    "lb_route_topk": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p],
+    "lb_route_topk": [c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    "lb_streams_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                        c_void_p, c_int, c_float, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
+    "lb_latent_rope": [c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
+                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
     "lb_expert_dispatch": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p],
     "lb_expert_gemm": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_longlong,
                        c_longlong, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p],
@@ -65,19 +69,19 @@ _SIGNATURES = {
     "lb_gated_recurrence": [c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "lb_gemm_heads_mma": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong,
-                          c_longlong, c_longlong, c_void_p, c_longlong, c_void_p],
+                          c_longlong, c_longlong, c_void_p, c_longlong, c_int, c_void_p],
     "lb_gemm_plain_batched": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_longlong,
-                              c_longlong, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong, c_void_p],
+                              c_longlong, c_longlong, c_longlong, c_longlong, c_void_p, c_longlong, c_int, c_void_p],
     "lb_add_rmsnorm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
     "lb_rope_kv": [c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_longlong, c_longlong, c_void_p, c_void_p,
                    c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int, c_void_p],
+                   c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_void_p],
     "lb_rotate_rows": [c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_int, c_float, c_int, c_int,
                        c_float, c_void_p],
     "lb_round_cols": [c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_void_p],
     "lb_attention_plain": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_float, c_void_p, c_int,
-                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
+                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "lb_short_conv": [c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_int, c_void_p],
     "lb_short_conv_state": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
@@ -276,21 +280,32 @@ def gated_recurrence(pre: torch.Tensor, q_col: int, f_col: int, v_col: int, bias
 
 def gemm_heads(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, gate: torch.Tensor | None = None) -> None:
     """y[t, h, :] = x[t, h, :] . w[h]^T for w [heads, N, K], one product a head, 32-bit sums: bfloat16 operands with K
-    a multiple of 8 on the tensor cores, everything else on the ordinary pipes.
-    With `gate` (float32 [T, >= heads * N], row-strided): y[t, h, n] *= sigmoid(gate[t, h * N + n]) before the rounding."""
+    a multiple of 8 on the tensor cores, everything else on the ordinary pipes.  x and y may be parts of longer heads
+    ([T, H, K] views with unit last stride).
+    With `gate` (float32 [T, heads * N], row-strided): y[t, h, n] *= sigmoid(gate[t, h * N + n]) before the rounding; a
+    gate of [T, heads] is one number a head."""
     T, H, K = x.shape
     N = w.shape[1]
-    _check(x, "x"); _check(w, "per-head weights"); _check(y, "y")
+    _check(w, "per-head weights")
+    for t, what in ((x, "x"), (y, "y")):
+        if not t.is_cuda or t.stride(2) != 1:
+            raise KernelError(f"{what} must be on the GPU with unit stride in its last dimension")
     if tuple(w.shape) != (H, N, K) or tuple(y.shape) != (T, H, N):
         raise KernelError(f"per-head product shapes do not fit: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
-    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] != H * N):
-        raise KernelError("the gate must be float32 [T, heads * N] with unit column stride")
-    if (x.dtype == w.dtype == y.dtype == torch.bfloat16 and K % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0):
-        _call("lb_gemm_heads_mma", y.data_ptr(), x.data_ptr(), w.data_ptr(), H, T, N, K, H * K, H * N, K, N * K, N, _ptr(gate),
-              gate.stride(0) if gate is not None else 0, stream)
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or gate.shape[0] != T or gate.shape[1] not in (H, H * N)):
+        raise KernelError("the gate must be float32 [T, heads * N] or [T, heads] with unit column stride")
+    one = 1 if gate is not None and gate.shape[1] == H else 0
+    if T == 0:
+        return
+    bx, by = x.stride(1), y.stride(1)
+    ldx, ldy = (x.stride(0), y.stride(0)) if T > 1 else (max(x.stride(0), H * bx), max(y.stride(0), H * by))
+    if (x.dtype == w.dtype == y.dtype == torch.bfloat16 and K % 8 == 0 and ldx % 8 == 0 and bx % 8 == 0 and x.data_ptr() % 16 == 0
+            and w.data_ptr() % 16 == 0):
+        _call("lb_gemm_heads_mma", y.data_ptr(), x.data_ptr(), w.data_ptr(), H, T, N, K, ldx, ldy, bx, N * K, by, _ptr(gate),
+              gate.stride(0) if gate is not None else 0, one, stream)
         return
     _call("lb_gemm_plain_batched", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), dtype_code(x.dtype), w.data_ptr(),
-          dtype_code(w.dtype), H, T, N, K, H * K, H * N, K, N * K, N, _ptr(gate), gate.stride(0) if gate is not None else 0, stream)
+          dtype_code(w.dtype), H, T, N, K, ldx, ldy, bx, N * K, by, _ptr(gate), gate.stride(0) if gate is not None else 0, one, stream)
 
 
 def add_rmsnorm(out: torch.Tensor, residual: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor,
@@ -366,6 +381,75 @@ def stream_norm(residual: torch.Tensor, stream: int, out: torch.Tensor | None = 
           n, H, stream)
 
 
+def streams_norm(out: torch.Tensor, x: torch.Tensor, streams: int, weight: torch.Tensor, eps: float, stream: int,
+                 read: torch.Tensor | None = None, update: tuple | None = None, x_new: torch.Tensor | None = None,
+                 rows: torch.Tensor | None = None) -> None:
+    """One pass between two sublayers of a model with `streams` = S parallel residual streams, in 32-bit.  x: [T, S, H], or
+    [T, H] when all streams are that one row.  `update` = (mix [S, S], out [S], y): x_t <- sum_s mix[s, t] x_s + out[t] y with
+    y a sublayer's output [T, H] (float32 or bfloat16), or (expert rows [places, H] float32, place_of [T * top], weights [T, top]
+    or one number), whose weighted sum is meant; the new streams go to x_new ([T, S, H], may be x) if given.  Then
+    u = sum_t read[t] x_t (without `read` the plain sum) and out = u / sqrt(mean(u^2) + eps) * weight, on `rows` if given."""
+    _check(out, "norm output"); _check(x, "streams", torch.float32); _check(weight, "norm weight", torch.float32)
+    H, T = x.shape[-1], x.shape[0]
+    same = x.dim() == 2
+    if (not same and tuple(x.shape) != (T, streams, H)) or weight.numel() != H:
+        raise KernelError(f"{tuple(x.shape)} are not {streams} streams, or the norm weight has not their size")
+    if x_new is not None:
+        _check(x_new, "new streams", torch.float32)
+        if tuple(x_new.shape) != (T, streams, H):
+            raise KernelError("the new streams are [T, streams, hidden]")
+    if rows is not None:
+        _check(rows, "row index", torch.int32)
+    n = T if rows is None else rows.shape[0]
+    if tuple(out.shape) != (n, H):
+        raise KernelError(f"an output of {tuple(out.shape)} for {n} rows of {H}")
+    mix = to = y = e = place_of = weights = None
+    top, w1 = 0, 0.0
+    if read is not None:
+        _check(read, "read weights", torch.float32)
+    if update is not None:
+        mix, to, y = update
+        _check(mix, "mix", torch.float32); _check(to, "write weights", torch.float32)
+        if mix.numel() != streams * streams or to.numel() != streams:
+            raise KernelError("the mix is [streams, streams], the write weights [streams]")
+        if isinstance(y, tuple):
+            e, place_of, weights = y
+            y = None
+            _check(e, "experts' rows", torch.float32); _check(place_of, "places", torch.int32)
+            top = place_of.numel() // T if T else 1
+            if torch.is_tensor(weights):
+                _check(weights, "expert weights", torch.float32)
+            else:
+                weights, w1 = None, float(weights)
+        else:
+            _check(y, "sublayer output")
+            if tuple(y.shape) != (T, H):
+                raise KernelError("a sublayer's output is [T, hidden]")
+    _call("lb_streams_norm", out.data_ptr(), dtype_code(out.dtype), x.data_ptr(), _ptr(x_new), streams, 1 if same else 0, _ptr(mix), _ptr(to),
+          _ptr(read), _ptr(y), dtype_code(y.dtype) if y is not None else F32, _ptr(e), _ptr(place_of), _ptr(weights), top, w1,
+          weight.data_ptr(), eps, _ptr(rows), n, H, stream)
+
+
+def latent_rope(pre: torch.Tensor, q_col: int, kv_col: int, heads: int, dim: int, rot: int, kv_rank: int, kv_w: torch.Tensor,
+                inv_freq: torch.Tensor | None, rot_dims: int, rot_scale: float, q_out: torch.Tensor, q_lat: torch.Tensor | None,
+                pages: torch.Tensor, step, block_table: torch.Tensor, page_size: int, eps: float, stream: int) -> None:
+    """From the float32 rows of `pre`: queries [heads x (dim | rot)] at q_col, their rot part rotated, to q_out [T, heads, dim + rot]
+    and, the rotated part alone, to q_lat [T, heads, kv_rank + rot] behind kv_rank places; the latent at kv_col, RMS-normed,
+    and the key part behind it, rotated, to the token's place in `pages` ([pages, 1, page_size, kv_rank + rot])."""
+    _rows32(pre, "input projections"); _check(kv_w, "latent norm", torch.float32); _check(q_out, "queries")
+    _check(pages, "latent pages", q_out.dtype); _check(block_table, "block table", torch.int32)
+    if inv_freq is not None:
+        _check(inv_freq, "frequencies", torch.float32)
+    T = pre.shape[0]
+    if tuple(q_out.shape) != (T, heads, dim + rot) or (q_lat is not None and tuple(q_lat.shape) != (T, heads, kv_rank + rot)):
+        raise KernelError("latent_rope: the outputs have the wrong shape")
+    if q_lat is not None:
+        _check(q_lat, "queries in latent space", q_out.dtype)
+    _call("lb_latent_rope", dtype_code(q_out.dtype), pre.data_ptr(), pre.stride(0), q_col, kv_col, heads, dim, rot, rot_dims, kv_rank,
+          kv_w.data_ptr(), _ptr(inv_freq), float(rot_scale), q_out.data_ptr(), _ptr(q_lat), pages.data_ptr(), step.positions.data_ptr(),
+          step.token_seq.data_ptr(), block_table.data_ptr(), T, page_size, block_table.shape[1], eps, stream)
+
+
 def rope_kv(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_out: torch.Tensor,
             positions: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, eps: float, stream: int,
             q_norm_w: torch.Tensor | None = None, k_norm_w: torch.Tensor | None = None,
@@ -373,14 +457,15 @@ def rope_kv(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_out: t
             k_cache: torch.Tensor | None = None, v_cache: torch.Tensor | None = None,
             token_seq: torch.Tensor | None = None, block_table: torch.Tensor | None = None, page_size: int = 0,
             k_out: torch.Tensor | None = None, v_out: torch.Tensor | None = None, v_dim: int = 0, rot_scale: float = 1.0,
-            pairs: bool = False, unit: bool = False) -> None:
+            pairs: bool = False, unit: bool = False, temperature: tuple | None = None) -> None:
     """Per-head norm of q and k, rotation, and the write of k and v into pages (or into k_out, v_out).
 
     q_in, k_in and v_in are 2-d views whose rows may be column ranges of one wider matrix; they may be float32 where
     the heads are stored in bfloat16 (a product with 32-bit output).  `v_dim`: the size of a value head if it is not
     head_dim (the value pool then has rows of that size).  `rot_scale` multiplies the rotation's sines and cosines.
     `pairs`: neighbours (2i, 2i + 1) are rotated together, not (i, i + rot_dim/2).  `unit`: behind the rotation every q and
-    k head is divided by sqrt(mean(x^2) + eps) (no norm weights then)."""
+    k head is divided by sqrt(mean(x^2) + eps) (no norm weights then).  `temperature` = (coef, every): behind all that the queries
+    at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
     T = q_in.shape[0]
     dt = q_out.dtype
     for t, w in ((q_in, "q"), (k_in, "k"), (v_in, "v")):
@@ -396,7 +481,7 @@ def rope_kv(q_in: torch.Tensor, k_in: torch.Tensor, v_in: torch.Tensor, q_out: t
           k_in.stride(0), v_in.stride(0), q_out.data_ptr(), _ptr(k_out), _ptr(v_out), _ptr(k_cache), _ptr(v_cache),
           positions.data_ptr(), _ptr(token_seq), _ptr(block_table), _ptr(q_norm_w), _ptr(k_norm_w), _ptr(inv_freq),
           T, num_q_heads, num_kv_heads, head_dim, rot_dim, page_size, max_pages, eps, dtype_code(q_in.dtype), v_dim, float(rot_scale),
-          1 if pairs else 0, 1 if unit else 0, stream)
+          1 if pairs else 0, 1 if unit else 0, float(temperature[0]) if temperature else 0.0, int(temperature[1]) if temperature else 0, stream)
 
 
 def rotate_rows(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor | None, head_dim: int, rot_dim: int, ranges,
@@ -428,8 +513,9 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
                     num_q_heads: int, num_kv_heads: int, head_dim: int, page_size: int, window: int, scale: float,
                     stream: int, v_dim: int = 0, slopes: torch.Tensor | None = None, softcap: float = 0.0,
                     sinks: torch.Tensor | None = None, pool: int = 0, pool_k: torch.Tensor | None = None,
-                    pool_v: torch.Tensor | None = None, pool_table: torch.Tensor | None = None, chunk: int = 0) -> None:
-    """`chunk` = C > 0: the query at position i sees the keys floor(i / C) * C .. i only.
+                    pool_v: torch.Tensor | None = None, pool_table: torch.Tensor | None = None, chunk: int = 0, v_stride: int = 0) -> None:
+    """`v_stride`: entries between the value pool's rows if not v_dim (values that are the first entries of longer rows).
+    `chunk` = C > 0: the query at position i sees the keys floor(i / C) * C .. i only.
     `v_dim`: the size of a value head if it is not head_dim (out is then [T, heads, v_dim]); `slopes` (float32
     [heads]): the score of key j for the query at position i is lowered by slopes[h] * (i - j).  `softcap` > 0: scores
     become softcap * tanh(score / softcap).  `sinks` (float32 [heads]): exp(sinks[h]) joins the softmax's denominator.
@@ -449,7 +535,7 @@ def attention_plain(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
           positions.data_ptr(), token_seq.data_ptr(), block_table.data_ptr(), q.shape[0], num_q_heads, num_kv_heads,
           head_dim, page_size, block_table.shape[1], window, scale, v_dim, _ptr(slopes), softcap, _ptr(sinks), pool,
           _ptr(pool_k) if pool else None, _ptr(pool_v) if pool else None, _ptr(pool_table) if pool else None,
-          pool_table.shape[1] if pool else 0, int(chunk), stream)
+          pool_table.shape[1] if pool else 0, int(chunk), int(v_stride), stream)
 
 
 def _rows32(t: torch.Tensor, what: str) -> None:
@@ -908,11 +994,12 @@ def head_gate(out: torch.Tensor, x: torch.Tensor, gate: torch.Tensor, scale: flo
 
 
 def route_topk(ids: torch.Tensor, weights: torch.Tensor, logits: torch.Tensor, correction: torch.Tensor | None, groups: int,
-               keep: int, scale: float, stream: int) -> None:
+               keep: int, scale: float, stream: int, softmax: bool = False) -> None:
     """The router's choice for every token: ids [T, top] int32 and weights [T, top] float32 from logits [T, experts]
     float32 (row-strided).  Scores are sigmoid(logits); chosen are the `top` largest of score + correction among the
     experts of the `keep` best of `groups` equal groups of neighbours (a group is worth its two largest); the weights
-    are the chosen plain scores over their sum (+ 1e-20), times scale."""
+    are the chosen plain scores over their sum (+ 1e-20), times scale.  `softmax`: the scores are the logits themselves (no
+    correction then) and the weights the softmax over the chosen ones, times scale."""
     _check(ids, "expert ids", torch.int32); _check(weights, "expert weights", torch.float32)
     if logits.dtype != torch.float32 or logits.stride(1) != 1:
         raise KernelError("the router's logits must be float32 with unit column stride")
@@ -920,7 +1007,7 @@ def route_topk(ids: torch.Tensor, weights: torch.Tensor, logits: torch.Tensor, c
         _check(correction, "correction", torch.float32)
     T, E = logits.shape
     _call("lb_route_topk", ids.data_ptr(), weights.data_ptr(), logits.data_ptr(), logits.stride(0) if T > 1 else E, _ptr(correction),
-          T, E, ids.shape[1], groups, keep, scale, stream)
+          T, E, ids.shape[1], groups, keep, scale, 1 if softmax else 0, stream)
 
 
 def expert_tile_rows(few: bool = False) -> int:

@@ -1,13 +1,14 @@
 from .base import (BatchShape, Block, FeedForward, KVCacheView, KVPages, Mixer, Norm, NormSink, ParamSpec, Part, PlanView,
                    PositionEncoding, RowScaled, Runtime, StateCacheView, StateSlot, StepContext, StepPlan)
-from .attention import CappedWindowAttention, GatedBiasAttention, GQAttention, distance_slopes
+from .attention import GatedBiasAttention, GQAttention, UnitHeadAttention, distance_slopes
 from .block import ParallelBlock, PostNormBlock, PreNormBlock, SandwichNormBlock
 from .causal_taps import CausalTaps
 from .decay_attention import DecayLinearAttention
 from .experts import RoutedExperts, TableExperts
 from .side_by_side import SideBySideMixer
 from .gated_recurrence import GatedLinearRecurrence
-from .latent_attention import LatentAttention
+from .hyper_connection import HyperConnection, HyperConnectionBlock
+from .latent_attention import LatentAttention, RotaryLatentAttention
 from .embedding import OutputHead, TokenEmbedding
 from .linear import Linear
 from .mlp import GatedFeedForward, SwiGLUFeedForward
@@ -21,5 +22,6 @@ __all__ = [
     "TokenEmbedding", "Linear", "SwiGLUFeedForward", "RMSNorm", "RotaryEmbedding", "ParallelBlock", "CausalTaps",
     "GatedLinearRecurrence", "LatentAttention", "GatedFeedForward", "GroupRMSNorm", "GatedBiasAttention", "distance_slopes",
     "PostNormBlock", "DecayLinearAttention", "RoutedExperts", "SideBySideMixer", "LayerNorm",
-    "CappedWindowAttention", "SandwichNormBlock", "TableExperts", "NeighbourRotary", "StreamEntry",
+    "UnitHeadAttention", "SandwichNormBlock", "TableExperts", "NeighbourRotary", "StreamEntry", "HyperConnection", "HyperConnectionBlock",
+    "RotaryLatentAttention",
 ]

@@ -581,22 +581,25 @@ class GatedWindowAttention(Mixer):
         return self.o.forward(inner, out_dtype=self.out_dtype)
 
 
-class CappedWindowAttention(Mixer):
-    """Softmax attention over a sliding window with a capped score, on heads whose queries and keys have unit mean square:
+class UnitHeadAttention(Mixer):
+    """Softmax attention on heads whose queries and keys have unit mean square, optionally over a sliding window, with a capped
+    score, a temperature of the query that grows with its position, and a gate of one number a head:
 
         q = unit(rotate(W_q x))      k = unit(rotate(W_k x))      v = W_v x        unit(z) = z / sqrt(mean(z^2) + eps), per head
-            (rotation of the first rot_dims entries of a head in pairs of neighbours; no weight in the norm behind it)
+            (rotation of the first rot_dims entries of a head in pairs of neighbours, or none; no weight in the norm behind it)
+        q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)     (`temperature` = (coef, every); None: not)
         the query at position i sees the keys j with 0 <= i - j < window (window 0: every j <= i)
-        out = softmax(softcap * tanh(q . k * scale / softcap)) v            (softcap 0: the scores as they are)
+        out_h = softmax(softcap * tanh(q . k * scale / softcap)) v            (softcap 0: the scores as they are)
+                [* sigmoid(W_g x)_h with `head_gate`]
 
-    Values may have another size than keys.  W_q | W_k | W_v are one product with 32-bit output; one kernel rotates, norms
-    and writes keys and values into their pages.  Beside forward(), the mixer offers its steps apart (in_names / in_sizes,
+    Values may have another size than keys.  W_q | W_k | W_v [| W_g] are one product with 32-bit output; one kernel rotates,
+    norms and writes keys and values into their pages.  Beside forward(), the mixer offers its steps apart (in_names / in_sizes,
     inner, `o`)."""
     recordable = True
 
     def __init__(self, rt: Runtime, prefix: str, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float,
                  softcap: float, position_encoding: Optional[NeighbourRotary], window: int, eps: float,
-                 out_dtype: Optional[torch.dtype] = None):
+                 out_dtype: Optional[torch.dtype] = None, head_gate: bool = False, temperature: Optional[tuple] = None):
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads are not a multiple of {kv_heads} kv heads")
         if position_encoding is not None and not hasattr(position_encoding, "pair_table"):
@@ -605,15 +608,18 @@ class CappedWindowAttention(Mixer):
         self.heads, self.kv_heads, self.dim, self.vdim = heads, kv_heads, dim, vdim
         self.scale, self.softcap, self.window, self.eps = float(scale), float(softcap), int(window), float(eps)
         self.position_encoding, self.out_dtype = position_encoding, out_dtype
+        self.head_gate = bool(head_gate)
+        self.temperature = (float(temperature[0]), int(temperature[1])) if temperature is not None else None
         self.q_size, self.k_size, self.v_size, self.inner_size = heads * dim, kv_heads * dim, kv_heads * vdim, heads * vdim
         self.proj = Linear(rt, self.in_names(), width, self.in_sizes())
         self.o = Linear(rt, f"{prefix}.o", self.inner_size, width)
 
     def in_names(self) -> list[str]:
-        return [f"{self.prefix}.q", f"{self.prefix}.k", f"{self.prefix}.v"]
+        p = self.prefix
+        return [f"{p}.q", f"{p}.k", f"{p}.v"] + ([f"{p}.g"] if self.head_gate else [])
 
     def in_sizes(self) -> list[int]:
-        return [self.q_size, self.k_size, self.v_size]
+        return [self.q_size, self.k_size, self.v_size] + ([self.heads] if self.head_gate else [])
 
     def children(self) -> list[Part]:
         return [self.proj, self.o]
@@ -629,10 +635,10 @@ class CappedWindowAttention(Mixer):
 
     def inner(self, pre: torch.Tensor, step: StepContext, cache: KVCacheView, out: torch.Tensor, out_scale: float = 1.0,
               write_cache: bool = True) -> None:
-        """pre: float32 [T, >= sum(in_sizes())], the columns q | k | v of this mixer; out: [T, inner_size] in the activation
-        type (contiguous) receives the heads."""
-        if out_scale != 1.0 or not out.is_contiguous():
-            raise ops.KernelError("this attention writes unscaled heads into a matrix of their own")
+        """pre: float32 [T, >= sum(in_sizes())], the columns q | k | v [| g] of this mixer; out: [T, inner_size] in the activation
+        type (contiguous, and with out_scale 1, unless there is a gate) receives the heads."""
+        if not self.head_gate and (out_scale != 1.0 or not out.is_contiguous()):
+            raise ops.KernelError("this attention without a gate writes unscaled heads into a matrix of their own")
         rt = self.rt
         T, H, G, D, V = pre.shape[0], self.heads, self.kv_heads, self.dim, self.vdim
         c1, c2, c3 = self.q_size, self.q_size + self.k_size, self.q_size + self.k_size + self.v_size
@@ -640,10 +646,15 @@ class CappedWindowAttention(Mixer):
         q = rt.empty((T, H, D))
         ops.rope_kv(pre[:, :c1], pre[:, c1:c2], pre[:, c2:c3], q, step.positions, H, G if write_cache else 0, D, self.eps, rt.stream,
                     inv_freq=inv_freq, rot_dim=rot, k_cache=cache.k, v_cache=cache.v, token_seq=step.token_seq,
-                    block_table=step.block_tables[cache.group], page_size=cache.page_size, v_dim=V, pairs=True, unit=True)
-        ops.attention(q, out.view(T, H, V), cache.k, cache.v, step, cache.group, H, G, D, cache.page_size, self.window, self.scale,
+                    block_table=step.block_tables[cache.group], page_size=cache.page_size, v_dim=V, pairs=True, unit=True,
+                    temperature=self.temperature)
+        heads = rt.empty((T, H, V)) if self.head_gate else out.view(T, H, V)
+        # |q| and |k| are at most sqrt(D), but for their rounding to 16 bits (and a temperature of the query)
+        ops.attention(q, heads, cache.k, cache.v, step, cache.group, H, G, D, cache.page_size, self.window, self.scale,
                       rt.stream, plan=step.plans.get(self.plan_key()), v_dim=V if V != D else 0, softcap=self.softcap,
-                      score_bound=1.02 * D)           # |q| and |k| are at most sqrt(D), but for their rounding to 16 bits
+                      score_bound=1.02 * D if self.temperature is None else 0.0)
+        if self.head_gate:
+            ops.head_gate(out, heads, pre[:, c3:c3 + H], out_scale, rt.stream)
 
     def forward(self, h: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
         pre = self.proj.forward(h, out_dtype=torch.float32)

@@ -38,7 +38,7 @@ import torch
 class ParamSpec:
     name: str                       # full tensor name in the checkpoint
     shape: tuple[int, ...]
-    init: str = "linear"            # "linear" | "embedding" | "norm" | "unit": how random weights are drawn
+    init: str = "linear"            # "linear" | "embedding" | "norm" | "norm0" | "unit" | "ones": how random weights are drawn
     integer: bool = False           # integer tables are kept as int32
     below: int = 0                  # integer tables: how random ones are drawn, rows of distinct numbers 0 .. below - 1 (0: any numbers)
 
@@ -193,6 +193,16 @@ class Pending:
 
 
 @dataclass
+class StreamUpdate:
+    """What a block hands on as `delta` when the model keeps several residual streams and the last sublayer's output is still to
+    be written into them: the output (a tensor, or ExpertSum) and the connection that says how (parts/hyper_connection.py).
+    The norm that reads the streams next does both in its pass (Norm.takes_streams); `residual` is then [T, streams, width],
+    or [T, width] as long as all streams are one row."""
+    output: Any
+    connection: Any
+
+
+@dataclass
 class ExpertSum:
     """The output of routed experts that is not summed yet: out[t] = sum_k weights[t, k] rows[place_of[t, k]] (+ the output
     of the expert every token uses, times sigmoid(gate_weight . gate_input[t]) if there is a gate)."""
@@ -261,6 +271,8 @@ class Norm(Part):
     takes_delta_parts = False
     # True: add_forward() also takes a Pending as `delta`.
     takes_pending = False
+    # True: add_forward() also takes a StreamUpdate as `delta` (the sum of the streams is normed then), and read_streams() is there.
+    takes_streams = False
 
     def add_forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], out_dtype: torch.dtype,
                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -331,6 +343,7 @@ class Block(Part):
     takes_delta_parts = False       # True: forward() takes such a tuple as `delta` (its first norm adds both)
     takes_stream_copy = False       # True: forward() takes a StreamCopy as `delta` (see there)
     takes_pending = False           # True: forward() takes a Pending as `delta`
+    takes_streams = False           # True: forward() takes a StreamUpdate as `delta`
 
     def cache_request(self) -> KVPages | StateSlot | None | tuple:
         """What a call of this block keeps of past tokens: the mixer's cache, unless the block has state of its own

@@ -6,6 +6,7 @@ RoutedExperts chooses by a router:
     experts form `groups` equal groups of neighbours; a group is worth the sum of its two largest c; only experts of the
     `keep` best groups can be chosen; the `top` experts with the largest c are
     weights = s of the chosen / (their sum + 1e-20) * scale          (the correction steers the choice only)
+    or, with `scores="softmax"`: c = z, and the weights are the softmax over the chosen z alone, times scale
     out = sum_k weight_k * expert_k(h) [+ shared(h)]
 
 TableExperts has no router: a table [vocab, top] names the experts of every token id, and each counts 1 / top,
@@ -132,13 +133,16 @@ class ExpertBank(FeedForward):
 class RoutedExperts(ExpertBank):
     def __init__(self, rt: Runtime, prefix: str, width: int, experts: int, top: int, ff: int, act: str, limit: float,
                  router_scale: float, groups: int = 1, keep: int = 1, shared: Optional[FeedForward] = None,
-                 correction: bool = True, out_dtype: Optional[torch.dtype] = None):
+                 correction: bool = True, out_dtype: Optional[torch.dtype] = None, scores: str = "sigmoid"):
+        if scores not in ("sigmoid", "softmax") or (scores == "softmax" and correction):
+            raise ValueError(f"scores {scores!r}: sigmoid, or softmax without a correction")
         if experts % groups or not (0 < keep <= groups) or not (0 < top <= keep * (experts // groups)):
             raise ValueError(f"{experts} experts, top {top}, {groups} groups of which {keep} are kept do not fit")
         super().__init__(rt, prefix, width, experts, top, ff, act, limit)
         self.router_scale, self.groups, self.keep = float(router_scale), groups, keep
         self.shared, self.has_correction = shared, correction
         self.out_dtype = out_dtype          # type of the result (None: the activation type)
+        self.scores = scores
         self.router = Linear(rt, f"{prefix}.router", width, experts)
         self.correction: torch.Tensor | None = None
 
@@ -154,15 +158,20 @@ class RoutedExperts(ExpertBank):
             self.correction = get(f"{self.prefix}.correction").to(torch.float32).contiguous()
         self.bind_experts(get)
 
-    def forward(self, h: torch.Tensor, step: StepContext) -> torch.Tensor:
+    offers_unsummed = True
+
+    def forward(self, h: torch.Tensor, step: StepContext, unsummed: bool = False):
         rt, top = self.rt, self.top
         T = h.shape[0]
         logits = self.router.forward(h, out_dtype=torch.float32)
         ids, weights = rt.empty((T, top), torch.int32), rt.empty((T, top), torch.float32)
-        ops.route_topk(ids, weights, logits, self.correction, self.groups, self.keep, self.router_scale, rt.stream)
+        ops.route_topk(ids, weights, logits, self.correction, self.groups, self.keep, self.router_scale, rt.stream,
+                       softmax=self.scores == "softmax")
         always = self.shared.forward(h, step) if self.shared is not None else None
         d = self.dispatch(ids, T)
         y = self.products(h, d)
+        if unsummed:
+            return ExpertSum(y, d.place_of, weights, always)
         out = rt.empty((T, self.width), self.out_dtype)
         ops.expert_combine(out, y, weights, d.place_of, rt.stream, always=always)
         return out

@@ -27,7 +27,7 @@ import torch
 
 from .. import ops
 from .attention import DECODE_ROWS, TILE_ROWS, plan_tiles
-from .base import BatchShape, KVCacheView, KVPages, Mixer, ParamSpec, Part, Runtime, StepContext, StepPlan
+from .base import BatchShape, KVCacheView, KVPages, Mixer, ParamSpec, Part, PositionEncoding, Runtime, StepContext, StepPlan
 from .linear import Linear
 
 
@@ -132,3 +132,75 @@ class LatentAttention(Mixer):
         gated = rt.empty((T, H, self.vdim))
         ops.gemm_heads(gated, mix, self.uv, rt.stream, gate=pre[:, self.q_rank + self.kv_rank:])
         return self.o.forward(gated.view(T, H * self.vdim))
+
+
+class RotaryLatentAttention(Mixer):
+    """Latent attention whose keys carry a rotated part that all heads share, with a learned sink and a gate of one number a head:
+
+        q_h = [q_u,h | rotate(q_r,h)]      from W_q u, head by head (dim | rot_dim entries)
+        c = rmsnorm(.) * w (kv_rank entries),  k_r = rotate(.) (rot_dim entries)      from W_dkv u
+        k_h = [W_uk[h] c | k_r],  v_h = W_uv[h] c
+        w_j = exp(q_h . k_h,j * scale) / (exp(sink_h) + sum_j<=i exp(q_h . k_h,j * scale))
+        out = W_o concat_h( sigmoid(W_g u)_h * sum_j w_j v_h,j )
+
+    [c | k_r] is all that is cached: one vector of kv_rank + rot_dim entries a token, key and value of one "head" whose values
+    are the first kv_rank entries (KVPages(1, kv_rank + rot_dim, shared=True)).  As in LatentAttention the head's key map
+    moves to the query and its value map behind the sum: attention runs as `heads` query heads [W_uk[h]^T q_u | q_r] over
+    the cached vectors.  W_q | W_dkv | W_g are one product with 32-bit output; one kernel norms the latent, rotates, and
+    writes the pages and the queries."""
+    recordable = True
+
+    def __init__(self, rt: Runtime, prefix: str, width: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int,
+                 scale: float, position_encoding: Optional[PositionEncoding], eps: float, out_dtype: Optional[torch.dtype] = None):
+        if position_encoding is not None and position_encoding.rotary_table() is None:
+            raise ValueError("this attention rotates by a table of frequencies (rotary_table)")
+        self.rt, self.prefix, self.width = rt, prefix, width
+        self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank = heads, dim, rot_dim, vdim, kv_rank
+        self.scale, self.eps, self.out_dtype = float(scale), float(eps), out_dtype
+        self.position_encoding = position_encoding
+        self.key_size = kv_rank + rot_dim
+        self.proj = Linear(rt, [f"{prefix}.q", f"{prefix}.dkv", f"{prefix}.g"], width, [heads * (dim + rot_dim), self.key_size, heads])
+        self.o = Linear(rt, f"{prefix}.o", heads * vdim, width)
+        self.kv_norm_w: torch.Tensor | None = None
+        self.sinks: torch.Tensor | None = None
+        self.uk_t: torch.Tensor | None = None       # [heads, kv_rank, dim]: W_uk[h]^T, the key map moved to the query
+        self.uv: torch.Tensor | None = None         # [heads, vdim, kv_rank]
+
+    def children(self) -> list[Part]:
+        return [self.proj, self.o]
+
+    def param_specs(self) -> list[ParamSpec]:
+        p = self.prefix
+        return [ParamSpec(f"{p}.dkv.norm", (self.kv_rank,), "norm"), ParamSpec(f"{p}.uk", (self.heads * self.dim, self.kv_rank)),
+                ParamSpec(f"{p}.uv", (self.heads * self.vdim, self.kv_rank)), ParamSpec(f"{p}.sink", (self.heads,))]
+
+    def bind(self, get: Callable[[str], torch.Tensor]) -> None:
+        p = self.prefix
+        self.kv_norm_w = get(f"{p}.dkv.norm").to(torch.float32).contiguous()
+        self.sinks = get(f"{p}.sink").to(torch.float32).contiguous()
+        self.uk_t = get(f"{p}.uk").view(self.heads, self.dim, self.kv_rank).transpose(1, 2).contiguous()
+        self.uv = get(f"{p}.uv").view(self.heads, self.vdim, self.kv_rank).contiguous()
+
+    def cache_request(self) -> KVPages:
+        return KVPages(1, self.key_size, 0, shared=True)
+
+    def forward(self, u: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
+        rt = self.rt
+        T, H, L = u.shape[0], self.heads, self.kv_rank
+        if not write_cache:
+            raise ops.KernelError("latent attention always writes its own latents")
+        n_q = H * (self.dim + self.rot_dim)
+        pre = self.proj.forward(u, out_dtype=torch.float32)                  # q | dkv | g
+        gate = pre[:, n_q + self.key_size:]
+        inv_freq, rot = self.position_encoding.rotary_table() if self.position_encoding is not None else (None, 0)
+        q, q_lat = rt.empty((T, H, self.dim + self.rot_dim)), rt.empty((T, H, self.key_size))
+        ops.latent_rope(pre, 0, n_q, H, self.dim, self.rot_dim, L, self.kv_norm_w, inv_freq, rot,
+                        getattr(self.position_encoding, "magnitude", 1.0), q, q_lat, cache.k, step, step.block_tables[cache.group],
+                        cache.page_size, self.eps, rt.stream)
+        gated = rt.empty((T, H, self.vdim))
+        ops.gemm_heads(q_lat[:, :, :L], q[:, :, :self.dim], self.uk_t, rt.stream)       # the head's key map, applied to the query
+        mix = rt.empty((T, H, L))
+        ops.attention_plain(q_lat, mix, cache.k, cache.v, step.positions, step.token_seq, step.block_tables[cache.group], H, 1, self.key_size,
+                            cache.page_size, 0, self.scale, rt.stream, v_dim=L, v_stride=self.key_size, sinks=self.sinks)
+        ops.gemm_heads(gated, mix, self.uv, rt.stream, gate=gate)
+        return self.o.forward(gated.view(T, H * self.vdim), out_dtype=self.out_dtype)

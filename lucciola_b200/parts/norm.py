@@ -4,6 +4,9 @@
 GroupRMSNorm cuts the row into equal consecutive parts with a root mean square each; with one group it is the
 same function (it does not offer itself as a sink of a product's epilogue, which forms one sum a row).
 
+RMSNorm.read_streams() stands between the sublayers of a model that keeps several residual streams: it writes the last
+sublayer's output into them, forms what the next one reads and norms it, in one kernel.
+
 RMSNorm.add_forward() also takes a Pending: the terms still to be added to the stream, of which one may go through another
 RMSNorm first (models that norm what a sublayer returns as well as what the next one reads); one kernel forms both norms.
 
@@ -16,22 +19,25 @@ from typing import Callable, Optional
 import torch
 
 from .. import ops
-from .base import ExpertSum, Norm, NormSink, ParamSpec, Pending, Runtime
+from .base import ExpertSum, Norm, NormSink, ParamSpec, Pending, Runtime, StreamUpdate
 
 
 class RMSNorm(Norm):
+    """`around_zero`: the checkpoint stores the weight's distance from one."""
     recordable = True
 
-    def __init__(self, rt: Runtime, name: str, size: int, eps: float):
-        self.rt, self.name, self.size, self.eps = rt, name, size, float(eps)
+    def __init__(self, rt: Runtime, name: str, size: int, eps: float, around_zero: bool = False):
+        self.rt, self.name, self.size, self.eps, self.around_zero = rt, name, size, float(eps), bool(around_zero)
         self.weight: torch.Tensor | None = None     # float32 on the device
 
     def param_specs(self) -> list[ParamSpec]:
-        return [ParamSpec(self.name, (self.size,), "norm")]
+        return [ParamSpec(self.name, (self.size,), "norm0" if self.around_zero else "norm")]
 
     def bind(self, get: Callable[[str], torch.Tensor]) -> None:
         # bfloat16 -> float32 is exact; the kernels read norm weights as float32.
         self.weight = get(self.name).to(torch.float32).contiguous()
+        if self.around_zero:
+            self.weight = self.weight + 1.0
 
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         return self.add_forward(x, None, out_dtype)
@@ -40,9 +46,35 @@ class RMSNorm(Norm):
         return NormSink(residual, self.weight, self.eps)
 
     takes_pending = True
+    takes_streams = True
+
+    def read_streams(self, x: torch.Tensor, update: Optional[StreamUpdate], read: Optional[torch.Tensor], streams: int,
+                     out_dtype: torch.dtype, keep: bool = True, rows: Optional[torch.Tensor] = None) -> tuple[torch.Tensor, torch.Tensor]:
+        """(the streams behind `update`, this norm of what `read` [streams] makes of them; without `read` their sum) in one
+        pass over x: [T, streams, size], or [T, size] while all streams are that row.  Not `keep`: the new streams are not
+        written and x comes back as it was."""
+        out = self.rt.empty((x.shape[0] if rows is None else rows.shape[0], self.size), out_dtype)
+        x_new, terms = None, None
+        if update is not None:
+            y = update.output
+            if isinstance(y, ExpertSum):
+                if y.always is not None:
+                    total = self.rt.empty((x.shape[0], self.size), torch.float32)
+                    ops.expert_combine(total, y.rows, y.weights, y.place_of, self.rt.stream, always=y.always, gate_input=y.gate_input,
+                                       gate_weight=y.gate_weight)
+                    y = total
+                else:
+                    y = (y.rows, y.place_of, y.weights)
+            terms = (update.connection.mix, update.connection.write, y)
+            if keep and rows is None:
+                x_new = x if x.dim() == 3 else self.rt.empty((x.shape[0], streams, self.size), torch.float32)
+        ops.streams_norm(out, x, streams, self.weight, self.eps, self.rt.stream, read=read, update=terms, x_new=x_new, rows=rows)
+        return (x if x_new is None else x_new), out
 
     def add_forward(self, residual: torch.Tensor, delta, out_dtype: torch.dtype,
                     rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        if isinstance(delta, StreamUpdate):
+            return self.read_streams(residual, delta, None, delta.connection.streams, out_dtype, keep=False, rows=rows)[1]
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = self.rt.empty((n, self.size), out_dtype)
         if isinstance(delta, Pending):

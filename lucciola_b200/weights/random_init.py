@@ -1,6 +1,7 @@
 """Random weights: a model folder (config.json, model.safetensors) from a configuration and a seed.
 
-Linear maps and the embedding are drawn from N(0, std), norm weights from 1 + N(0, norm_std), bounds
+Linear maps and the embedding are drawn from N(0, std), norm weights from 1 + N(0, norm_std)
+(or, stored around zero, N(0, norm_std)), stream weights from 1 / streams + N(0, std), bounds
 ("unit") uniformly from (0, 1);
 each tensor has its own generator seeded by (seed, tensor name), so a tensor's values do not
 depend on which other tensors exist.  Values are rounded to the storage type once; whoever reads
@@ -39,6 +40,10 @@ def random_tensor(spec: ParamSpec, seed: int, std: float, norm_std: float, dtype
     x = torch.randn(spec.shape, generator=g, device=device, dtype=torch.float32)
     if spec.init == "norm":
         x = 1.0 + norm_std * x
+    elif spec.init == "norm0":                     # a norm weight stored as its distance from one
+        x = norm_std * x
+    elif spec.init == "ones":                      # the few numbers that weigh parallel streams
+        x = 1.0 / spec.shape[-1] + std * x
     else:
         x = std * x
     return x.to(dtype)
