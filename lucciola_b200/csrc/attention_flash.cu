@@ -24,7 +24,7 @@
 //
 // Head sizes: any multiple of 8 up to 128 (padded with zeros to 64 or 128 in shared memory), keys (and queries) and
 // values each their own.
-#include "common.cuh"
+#include "warp_mma.cuh"
 
 #include <cuda.h>
 #include <mutex>
@@ -42,7 +42,7 @@ struct FlashParams {
   const bf16* k_cache; const bf16* v_cache; // [pages, nkv, page_size, d] (values: v_dim)
   const int* positions;                     // [T]
   const int* block_table; int max_pages;    // [S, max_pages]
-  const int4* tiles;                        // {first token, tokens, request index, unused}
+  const int4* tiles;                        // {first token, tokens, request index, the request's tokens in this step before the first}
   float* part_o;                            // [tiles, nkv, splits, part_rows, d]
   float* part_ml;                           // [tiles, nkv, splits, part_rows, 2]
   int part_rows;                            // most query rows of any tile
@@ -63,31 +63,6 @@ struct FlashParams {
   const int* pool_table; int pool_max_pages;// in the same softmax and without a distance bias
   int chunk;                                // C > 0: a row at position i sees no key before floor(i / C) * C (positions in runs of C)
 };
-
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool valid) {
-  const int n = valid ? 16 : 0;             // 0: the 16 bytes are filled with zeros, nothing is read
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-  __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
-  return *reinterpret_cast<uint32_t*>(&v);
-}
 
 __device__ __forceinline__ void fa_cluster_sync() {
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -555,43 +530,9 @@ flash_attention_kernel(FlashParams p) {
 // end) is replaced by page 0, whose keys are masked all the same.
 constexpr int FD_THREADS = 160;
 constexpr int FD_STAGES = 3;
-constexpr unsigned long long FD_WAIT_CYCLES = 4000000000ull;
 enum { FD_ERR_FULL = 401, FD_ERR_EMPTY = 402 };
 __device__ int g_flash_decode_error = 0;
 
-__device__ __forceinline__ void fd_mbar_init(uint32_t bar, uint32_t count) {
-  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count));
-}
-__device__ __forceinline__ void fd_mbar_expect_tx(uint32_t bar, uint32_t bytes) {
-  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void fd_mbar_arrive(uint32_t bar) {
-  asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ bool fd_mbar_try_wait(uint32_t bar, uint32_t parity) {
-  uint32_t ok;
-  asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-               : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-  return ok != 0;
-}
-// Bounded: gives up after about two seconds, leaves a code for the host and tells the rest of the CTA.
-template <bool SLEEP>
-__device__ __forceinline__ bool fd_mbar_wait(uint32_t bar, uint32_t parity, volatile int* abort_flag, int code) {
-  if (fd_mbar_try_wait(bar, parity)) return true;
-  const long long t0 = clock64();
-  for (unsigned it = 1;; ++it) {
-    if (SLEEP) __nanosleep(64);
-    if (fd_mbar_try_wait(bar, parity)) return true;
-    if ((it & 255u) == 0u) {
-      if (*abort_flag) return false;
-      if ((unsigned long long)(clock64() - t0) > FD_WAIT_CYCLES) {
-        *abort_flag = code;
-        atomicCAS(&g_flash_decode_error, 0, code);
-        return false;
-      }
-    }
-  }
-}
 __device__ __forceinline__ void fd_tma_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
                ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
@@ -641,7 +582,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
   const int num_stages = kend > kbeg ? (kend - kbeg + FA_KEYS - 1) / FA_KEYS : 0;
 
   if (tid == 0) {
-    for (int s = 0; s < FD_STAGES; ++s) { fd_mbar_init(full(s), 1); fd_mbar_init(empty(s), 4); }
+    for (int s = 0; s < FD_STAGES; ++s) { mbar_init(full(s), 1); mbar_init(empty(s), 4); }
     abort_word = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -666,18 +607,18 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
     int row = row_of(0);                            // the tables were written before the step began
     auto fetch = [&](int st) {
       const int b = st % FD_STAGES;
-      if (lane == 0) fd_mbar_expect_tx(full(b), STAGE_BYTES);
+      if (lane == 0) mbar_expect_tx(full(b), STAGE_BYTES);
       __syncwarp();
       if (active) fd_tma_2d(base + b * STAGE_BYTES + dst_off, map, half * 64, row, full(b));
       row = row_of(st + 1);                         // looked up while the stage is awaited
     };
-    // Keys before this step's first token were written by earlier steps: the first stages of them are requested while
-    // the kernel ahead (which writes this step's keys and values) may still run.
+    // Keys before the request's first token of this step were written by earlier steps: the first stages of them are
+    // requested while the kernel ahead (which writes this step's keys and values) may still run.
     int st = 0;
-    for (; st < min(num_stages, FD_STAGES) && kbeg + (st + 1) * FA_KEYS <= pos0; ++st) fetch(st);
+    for (; st < min(num_stages, FD_STAGES) && kbeg + (st + 1) * FA_KEYS <= pos0 - tile.w; ++st) fetch(st);
     pdl_wait();
     for (; st < num_stages; ++st) {
-      if (!fd_mbar_wait<true>(empty(st % FD_STAGES), (uint32_t)((st / FD_STAGES) & 1) ^ 1u, abort_flag, FD_ERR_EMPTY)) break;
+      if (!mbar_wait<true>(empty(st % FD_STAGES), (uint32_t)((st / FD_STAGES) & 1) ^ 1u, abort_flag, &g_flash_decode_error, FD_ERR_EMPTY)) break;
       fetch(st);
     }
     if (p.cluster > 0) { fa_cluster_sync(); fa_cluster_sync(); }      // the cluster's barriers count every thread
@@ -723,7 +664,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
 
   for (int st = 0; st < num_stages; ++st) {
     const int b = st % FD_STAGES;
-    if (!fd_mbar_wait<false>(full(b), (uint32_t)((st / FD_STAGES) & 1), abort_flag, FD_ERR_FULL)) break;
+    if (!mbar_wait<false>(full(b), (uint32_t)((st / FD_STAGES) & 1), abort_flag, &g_flash_decode_error, FD_ERR_FULL)) break;
     const uint32_t kb = base + b * STAGE_BYTES, vb = kb + MAT_BYTES;
     const int kbase = kbeg + st * FA_KEYS;
 
@@ -816,7 +757,7 @@ flash_decode_tma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_c
       mma_bf16(o[db + 1], pf, b2, b3);
     }
     __syncwarp();
-    if (lane == 0) fd_mbar_arrive(empty(b));          // this warp has read the stage
+    if (lane == 0) mbar_arrive(empty(b));          // this warp has read the stage
   }
 
 #pragma unroll
@@ -985,7 +926,8 @@ LB_EXPORT long long lb_attention_flash_workspace(int num_tiles, int num_kv_heads
   return (long long)num_tiles * num_kv_heads * splits * part_rows * (head_dim + 2);
 }
 
-// q, out: [T, nq, d] bfloat16.  tiles: [num_tiles] of {first token, tokens, request index, 0} with
+// q, out: [T, nq, d] bfloat16.  tiles: [num_tiles] of {first token, tokens, request index, the request's tokens in this step
+// before the tile's first} with
 // tokens * (nq / nkv) <= part_rows <= 64.  workspace: float32, needed when splits > 1.
 // kv_share >= 1: the pools hold num_kv_heads / kv_share heads and kv head j reads pool head j / kv_share, so that
 // many query heads on one cached head can be cut into groups of at most 16 (the tiles of the decode kernels).

@@ -116,6 +116,8 @@ _SIGNATURES = {
     "lb_attention_tcgen05": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                              c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_longlong, c_void_p, c_float, c_int, c_void_p,
                              c_void_p],
+    "lb_latent_flash": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                        c_float, c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p],
     "lb_sample": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
 }
 
@@ -1158,8 +1160,9 @@ def device_error() -> int:
     lib.lb_device_error.restype = c_int
     lib.lb_attention_tcgen05_device_error.restype = c_int
     lib.lb_attention_flash_device_error.restype = c_int
+    lib.lb_latent_flash_device_error.restype = c_int
     return (int(lib.lb_device_error()) or int(lib.lb_attention_tcgen05_device_error())
-            or int(lib.lb_attention_flash_device_error()))
+            or int(lib.lb_attention_flash_device_error()) or int(lib.lb_latent_flash_device_error()))
 
 
 def linear(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, fast: bool, post: str | None = None, post_c: float = 0.0) -> None:
@@ -1257,7 +1260,8 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
                     slopes: torch.Tensor | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None, pool: int = 0,
                     pool_k: torch.Tensor | None = None, pool_v: torch.Tensor | None = None,
                     pool_table: torch.Tensor | None = None, chunk: int = 0, v_dim: int = 0) -> None:
-    """Tensor-core attention over pages.  tiles: int32 [n, 4] of (first token, tokens, request index, 0).
+    """Tensor-core attention over pages.  tiles: int32 [n, 4] of (first token, tokens, request index,
+    the request's tokens in this step before the first).
     `kv_share` > 1: the pools hold num_kv_heads / kv_share heads, and kv head j of this call reads pool head j // kv_share
     (many query heads on one cached head, cut into groups of at most 16 so that decoded tokens fit the decode kernel's tiles).
     `force_workspace` sends the partial results of the splits through the workspace and the combining
@@ -1291,6 +1295,50 @@ def attention_flash(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v
           -splits if force_workspace else splits, max_rows, _ptr(ws), ws_elems, kv_share, _ptr(slopes), softcap, _ptr(sinks),
           pool, _ptr(pool_k) if pool else None, _ptr(pool_v) if pool else None, _ptr(pool_table) if pool else None,
           pool_table.shape[1] if pool else 0, int(chunk), int(v_dim), stream)
+
+
+def latent_flash_ok(dk: int, dv: int, group: int, page_size: int) -> bool:
+    """The sizes of the kernel for many heads on one cached vector: keys of up to 576 entries whose first up to 512 are the
+    values (multiples of 8), at most 64 heads a tile, pages of 8 to 128 tokens."""
+    lib = library()
+    lib.lb_latent_flash_ok.restype = c_int
+    lib.lb_latent_flash_ok.argtypes = [c_int, c_int, c_int, c_int]
+    return bool(lib.lb_latent_flash_ok(dk, dv, group, page_size))
+
+
+def latent_flash_splits(num_tiles: int, head_groups: int, max_span: int, slots: int = 148) -> int:
+    """Into how many key ranges a launch is cut: the count that takes the fewest rounds of the SMs times keys a range, with the
+    CTAs' start and end worth 128 keys and the second kernel 192.  A range has 128 keys at least."""
+    ctas = max(num_tiles * head_groups, 1)
+    best, best_cost = 1, float("inf")
+    for s in range(1, min(32, max(1, max_span // 128)) + 1):
+        cost = -(-ctas * s // slots) * (128 + -(-max_span // s)) + (192 if s > 1 else 0)
+        if cost < best_cost - 1e-9:
+            best, best_cost = s, cost
+    return best
+
+
+def latent_flash(q: torch.Tensor, out: torch.Tensor, pool: torch.Tensor, positions: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor,
+                 max_rows: int, group: int, page_size: int, scale: float, splits: int, stream: int, sinks: torch.Tensor | None = None) -> None:
+    """Causal attention of q [T, heads, dk] over the cached vectors `pool` [pages, 1, page_size, dk], whose first dv entries are the
+    values: out [T, heads, dv].  tiles: int32 [n, 4] of (first token, tokens, request index, the request's tokens in
+    this step before the first) with tokens * group <= max_rows
+    <= 64; `group` heads share a tile.  `sinks` (float32 [heads]): exp(sinks[h]) joins the denominator."""
+    _check(q, "q", torch.bfloat16); _check(out, "attention output", torch.bfloat16); _check(pool, "latent pool", torch.bfloat16)
+    _check(positions, "positions", torch.int32); _check(block_table, "block table", torch.int32); _check(tiles, "tiles", torch.int32)
+    if sinks is not None:
+        _check(sinks, "sinks", torch.float32)
+    T, H, dk = q.shape
+    dv = out.shape[2]
+    if tuple(out.shape[:2]) != (T, H) or pool.shape[-1] != dk or (sinks is not None and sinks.numel() != H):
+        raise KernelError("latent attention: q, out, the pool and the sinks do not fit")
+    n = tiles.shape[0]
+    ws, elems = None, 0
+    if splits > 1:
+        ws = _attention_workspace(q.device, n * (H // group) * splits * max_rows * (dv + 2))
+        elems = ws.numel()
+    _call("lb_latent_flash", q.data_ptr(), out.data_ptr(), pool.data_ptr(), positions.data_ptr(), block_table.data_ptr(), tiles.data_ptr(),
+          n, H, group, dk, dv, page_size, block_table.shape[1], pool.shape[0], scale, _ptr(sinks), splits, max_rows, _ptr(ws), elems, stream)
 
 
 def attention_tcgen05_ok(q: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, page_size: int,
@@ -1356,7 +1404,7 @@ def attention_tcgen05(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                       key_splits: int = 1, slopes: torch.Tensor | None = None, softcap: float = 0.0,
                       score_bound: float = 0.0) -> None:
     """Attention of portions of prompts on tcgen05 (S and O in tensor memory).  tiles: int32 [n, 4] of
-    (first token, tokens, request index, 0) with tokens <= 2 * (128 // (nq // nkv)).  With key_splits > 1 the keys of
+    (first token, tokens, request index, unused) with tokens <= 2 * (128 // (nq // nkv)).  With key_splits > 1 the keys of
     every tile are cut into that many ranges, a CTA each, combined by a second kernel.
     `score_bound` > 0 with a cap: no |q . k| is larger (queries and keys of unit mean square, say); the kernel may then form
     the cap as a polynomial and leave the running maximum out."""

@@ -32,14 +32,14 @@ TILE_ROWS, DECODE_ROWS = 64, 16
 
 
 def tiles_of(q_lens: Sequence[int], group: int, rows: int, take=None) -> list[tuple[int, int, int, int]]:
-    """Runs of up to rows // group consecutive tokens of one request: (first token, tokens, request, 0),
-    for the requests whose number of tokens passes `take`."""
+    """Runs of up to rows // group consecutive tokens of one request: (first token, tokens, request, the request's tokens in
+    this step before the first), for the requests whose number of tokens passes `take`."""
     per = rows // group
     tiles, t = [], 0
     for i, n in enumerate(q_lens):
         if take is None or take(n):
             for off in range(0, n, per):
-                tiles.append((t + off, min(per, n - off), i, 0))
+                tiles.append((t + off, min(per, n - off), i, off))
         t += n
     return tiles
 

@@ -23,10 +23,11 @@ from __future__ import annotations
 
 from typing import Callable, Hashable, Optional
 
+import numpy as np
 import torch
 
 from .. import ops
-from .attention import DECODE_ROWS, TILE_ROWS, plan_tiles
+from .attention import DECODE_ROWS, TILE_ROWS, plan_tiles, tiles_of
 from .base import BatchShape, KVCacheView, KVPages, Mixer, ParamSpec, Part, PositionEncoding, Runtime, StepContext, StepPlan
 from .linear import Linear
 
@@ -184,6 +185,34 @@ class RotaryLatentAttention(Mixer):
     def cache_request(self) -> KVPages:
         return KVPages(1, self.key_size, 0, shared=True)
 
+    @property
+    def group(self) -> int:
+        """Heads that share a tile of query rows: all of them up to 64, else their largest equal groups of at most 64."""
+        return next(self.heads // s for s in range(1, self.heads + 1) if self.heads % s == 0 and self.heads // s <= TILE_ROWS)
+
+    def plan_key(self) -> Optional[Hashable]:
+        return ("latent tiles", self.group) if self.rt.fast_kernels and self.scale > 0 else None
+
+    def plan(self, batch: BatchShape) -> Optional[StepPlan]:
+        """Tiles of up to 64 query rows; where single tokens are in the step, tiles of as few rows as one token needs (the
+        kernel's work follows the largest tile)."""
+        g = self.group
+        rows = -(-g // 16) * 16 if 1 in batch.q_lens else TILE_ROWS
+        tiles = tiles_of(batch.q_lens, g, rows)
+        return StepPlan({"all": np.asarray(tiles, dtype=np.int32).reshape(len(tiles), 4)}, {"rows": {"all": max(n for _, n, _, _ in tiles) * g}})
+
+    def _attend(self, q_lat: torch.Tensor, mix: torch.Tensor, step: StepContext, cache: KVCacheView) -> None:
+        table = step.block_tables[cache.group]
+        plan = step.plans.get(self.plan_key())
+        if plan is None or not ops.latent_flash_ok(self.key_size, self.kv_rank, self.group, cache.page_size):
+            ops.attention_plain(q_lat, mix, cache.k, cache.v, step.positions, step.token_seq, table, self.heads, 1, self.key_size,
+                                cache.page_size, 0, self.scale, self.rt.stream, v_dim=self.kv_rank, v_stride=self.key_size, sinks=self.sinks)
+            return
+        tiles = plan.arrays["all"]
+        splits = ops.latent_flash_splits(tiles.shape[0], self.heads // self.group, step.span_hint or step.max_context_len)
+        ops.latent_flash(q_lat, mix, cache.k, step.positions, table, tiles, plan.host["rows"]["all"], self.group, cache.page_size, self.scale,
+                         splits, self.rt.stream, sinks=self.sinks)
+
     def forward(self, u: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
         rt = self.rt
         T, H, L = u.shape[0], self.heads, self.kv_rank
@@ -200,7 +229,6 @@ class RotaryLatentAttention(Mixer):
         gated = rt.empty((T, H, self.vdim))
         ops.gemm_heads(q_lat[:, :, :L], q[:, :, :self.dim], self.uk_t, rt.stream)       # the head's key map, applied to the query
         mix = rt.empty((T, H, L))
-        ops.attention_plain(q_lat, mix, cache.k, cache.v, step.positions, step.token_seq, step.block_tables[cache.group], H, 1, self.key_size,
-                            cache.page_size, 0, self.scale, rt.stream, v_dim=L, v_stride=self.key_size, sinks=self.sinks)
+        self._attend(q_lat, mix, step, cache)
         ops.gemm_heads(gated, mix, self.uv, rt.stream, gate=gate)
         return self.o.forward(gated.view(T, H * self.vdim), out_dtype=self.out_dtype)

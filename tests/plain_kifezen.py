@@ -88,18 +88,15 @@ def rotate_halves(x: torch.Tensor, positions: torch.Tensor, rot) -> torch.Tensor
 def causal_softmax_attention(q, k, v, start: int, scale: float, sinks=None):
     """q [T, H, D] at positions start .. over keys k [n, G, D] and values v [n, G, V] at positions 0 .. n - 1; with `sinks`
     [H] the denominator of head h also holds exp(sinks[h])."""
-    T, H, _ = q.shape
+    T, H, D = q.shape
     G, V = k.shape[1], v.shape[2]
-    per = H // G
     out = torch.zeros(T, H, V, dtype=q.dtype)
     for t in range(T):
-        i = start + t
-        for g in range(G):
-            s = (q[t, g * per:(g + 1) * per] @ k[:i + 1, g].T) * scale
-            if sinks is not None:
-                s = torch.cat([s, sinks[g * per:(g + 1) * per, None].to(s.dtype)], dim=-1)
-            w = torch.softmax(s, dim=-1)[:, :i + 1]
-            out[t, g * per:(g + 1) * per] = w @ v[:i + 1, g]
+        n = start + t + 1
+        s = q[t].reshape(G, H // G, D) @ k[:n].permute(1, 2, 0) * scale                          # [G, H / G, n]
+        if sinks is not None:
+            s = torch.cat([s, sinks.to(s.dtype).reshape(G, H // G, 1)], dim=-1)
+        out[t] = (torch.softmax(s, dim=-1)[..., :n] @ v[:n].permute(1, 0, 2)).reshape(H, V)
     return out
 
 
