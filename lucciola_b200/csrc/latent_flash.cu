@@ -129,6 +129,9 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
       if (!mbar_wait<true>(empty(st % STAGES), (uint32_t)((st / STAGES) & 1) ^ 1u, &abort_word[1], &g_latent_flash_error, LF_ERR_EMPTY)) break;
       fetch(st);
     }
+    // nobody leaves while a copy of its own is in flight
+    for (int j = max(0, st - STAGES); j < st; ++j)
+      mbar_wait<true>(full(j % STAGES), (uint32_t)((j / STAGES) & 1), &abort_word[1], &g_latent_flash_error, LF_ERR_FULL);
     return;
   }
 

@@ -118,6 +118,9 @@ _SIGNATURES = {
                              c_void_p],
     "lb_latent_flash": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_float, c_void_p, c_int, c_int, c_void_p, c_longlong, c_void_p],
+    "lb_latent_gather": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "lb_latent_prefill": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                          c_float, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p],
     "lb_sample": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
 }
 
@@ -1161,8 +1164,10 @@ def device_error() -> int:
     lib.lb_attention_tcgen05_device_error.restype = c_int
     lib.lb_attention_flash_device_error.restype = c_int
     lib.lb_latent_flash_device_error.restype = c_int
+    lib.lb_latent_prefill_device_error.restype = c_int
     return (int(lib.lb_device_error()) or int(lib.lb_attention_tcgen05_device_error())
-            or int(lib.lb_attention_flash_device_error()) or int(lib.lb_latent_flash_device_error()))
+            or int(lib.lb_attention_flash_device_error()) or int(lib.lb_latent_flash_device_error())
+            or int(lib.lb_latent_prefill_device_error()))
 
 
 def linear(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, stream: int, fast: bool, post: str | None = None, post_c: float = 0.0) -> None:
@@ -1339,6 +1344,63 @@ def latent_flash(q: torch.Tensor, out: torch.Tensor, pool: torch.Tensor, positio
         elems = ws.numel()
     _call("lb_latent_flash", q.data_ptr(), out.data_ptr(), pool.data_ptr(), positions.data_ptr(), block_table.data_ptr(), tiles.data_ptr(),
           n, H, group, dk, dv, page_size, block_table.shape[1], pool.shape[0], scale, _ptr(sinks), splits, max_rows, _ptr(ws), elems, stream)
+
+
+def latent_prefill_ok(dim: int, rot: int, vdim: int, kv_rank: int) -> bool:
+    """The sizes of the tensor-memory kernel for latent attention with multiplied-out keys and values: heads of up to 128
+    unrotated and 64 rotated entries, values of up to 128, all sizes multiples of 8."""
+    return (0 < dim <= 128 and 0 <= rot <= 64 and 0 < vdim <= 128 and kv_rank > 0 and all(x % 8 == 0 for x in (dim, rot, vdim, kv_rank)))
+
+
+def latent_gather(out: torch.Tensor, pool: torch.Tensor, entries: torch.Tensor, context_lens: torch.Tensor, block_table: torch.Tensor,
+                  page_size: int, stream: int) -> None:
+    """out[first + j] = the cached vector of position j of a request, for `entries` int32 [n, 4] of (request index, first row, rows,
+    unused), whose rows lie one behind the other; zeros behind a request's last position.  pool [pages, 1, page_size, dk] bfloat16."""
+    _check(out, "gathered vectors", torch.bfloat16); _check(pool, "latent pool", torch.bfloat16); _check(entries, "entries", torch.int32)
+    _check(context_lens, "context lengths", torch.int32); _check(block_table, "block table", torch.int32)
+    if out.shape[1] != pool.shape[-1]:
+        raise KernelError("gathered vectors have the cached ones' size")
+    _call("lb_latent_gather", out.data_ptr(), pool.data_ptr(), entries.data_ptr(), entries.shape[0], out.shape[0], context_lens.data_ptr(),
+          block_table.data_ptr(), block_table.shape[1], page_size, out.shape[1], stream)
+
+
+def latent_prefill(q: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, lat: torch.Tensor, positions: torch.Tensor, tiles: torch.Tensor,
+                   dim: int, rot: int, kv_rank: int, scale: float, stream: int, sinks: torch.Tensor | None = None,
+                   gate: torch.Tensor | None = None, key_splits: int = 1) -> None:
+    """Causal attention of q [T, heads, dim + rot] over multiplied-out keys and values: kv [rows, heads * dim | heads * vdim], and the
+    rotated key part of all heads behind the first kv_rank entries of lat [rows, kv_rank + rot]; out [T, heads, vdim].  tiles:
+    int32 [n, 4] of (first token, tokens <= 256, unused, first row of its request), position j being row first + j.  `sinks`
+    (float32 [heads]): exp(sinks[h]) joins the denominator; `gate` (float32 [T, heads], row-strided): out *= sigmoid(gate)."""
+    for t, what in ((q, "q"), (out, "attention output"), (kv, "keys and values"), (lat, "gathered vectors")):
+        _check(t, what, torch.bfloat16)
+    _check(positions, "positions", torch.int32); _check(tiles, "tiles", torch.int32)
+    T, H, _ = q.shape
+    vdim = out.shape[2]
+    if (q.shape[2] != dim + rot or tuple(out.shape[:2]) != (T, H) or kv.shape[1] != H * (dim + vdim) or lat.shape[1] != kv_rank + rot
+            or lat.shape[0] != kv.shape[0]):
+        raise KernelError("latent prefill: q, out, the keys and values and the gathered vectors do not fit")
+    if gate is not None and (gate.dtype != torch.float32 or gate.stride(1) != 1 or tuple(gate.shape) != (T, H)):
+        raise KernelError("the gate must be float32 [T, heads] with unit column stride")
+    if sinks is not None:
+        _check(sinks, "sinks", torch.float32)
+    ws, elems = None, 0
+    if key_splits > 1:
+        ws = _attention_workspace(q.device, tiles.shape[0] * H * key_splits * 256 * (vdim + 2))
+        elems = ws.numel()
+    _call("lb_latent_prefill", q.data_ptr(), out.data_ptr(), kv.data_ptr(), lat.data_ptr(), positions.data_ptr(), tiles.data_ptr(), tiles.shape[0],
+          T, kv.shape[0], H, dim, rot, vdim, kv_rank, scale, _ptr(sinks), _ptr(gate), gate.stride(0) if gate is not None else 0, key_splits,
+          _ptr(ws), elems, stream)
+
+
+def latent_expansion_pays(tokens: int, span: int, heads: int, dim: int, rot: int, vdim: int, kv_rank: int) -> bool:
+    """Whether a portion of `tokens` tokens behind which lie up to `span` positions in all is done sooner with every head's keys and
+    values multiplied out of the latents (a product over `span` rows, then tensor-memory attention in tiles of 128 queries)
+    than by the kernel that leaves them in latent space.  By the operations of both and the rates the kernels reach; it depends
+    on the step's shape alone, so recordings keep it."""
+    seen = span - 0.5 * tokens
+    expanded = 2.0 * span * heads * (dim + vdim) * kv_rank / 1.0e15 + 2.0 * (-(-tokens // 128) * 128) * seen * heads * (dim + rot + vdim) / 4.5e14 + 8e-6
+    absorbed = 2.0 * tokens * seen * heads * (2 * kv_rank + rot) / 2.2e14 + 2.0 * tokens * heads * kv_rank * (dim + vdim) / 2.5e14
+    return expanded < absorbed
 
 
 def attention_tcgen05_ok(q: torch.Tensor, num_q_heads: int, num_kv_heads: int, head_dim: int, page_size: int,

@@ -27,9 +27,12 @@ import numpy as np
 import torch
 
 from .. import ops
-from .attention import DECODE_ROWS, TILE_ROWS, plan_tiles, tiles_of
+from .attention import BIG_PORTION, DECODE_ROWS, TILE_ROWS, plan_tiles, tiles_of
 from .base import BatchShape, KVCacheView, KVPages, Mixer, ParamSpec, Part, PositionEncoding, Runtime, StepContext, StepPlan
 from .linear import Linear
+
+# Most bytes that a step's multiplied-out keys and values may take; portions beyond are left in latent space.
+EXPANSION_BYTES = 1 << 30
 
 
 class LatentAttention(Mixer):
@@ -160,12 +163,14 @@ class RotaryLatentAttention(Mixer):
         self.scale, self.eps, self.out_dtype = float(scale), float(eps), out_dtype
         self.position_encoding = position_encoding
         self.key_size = kv_rank + rot_dim
+        self.expandable = ops.latent_prefill_ok(dim, rot_dim, vdim, kv_rank)
         self.proj = Linear(rt, [f"{prefix}.q", f"{prefix}.dkv", f"{prefix}.g"], width, [heads * (dim + rot_dim), self.key_size, heads])
         self.o = Linear(rt, f"{prefix}.o", heads * vdim, width)
         self.kv_norm_w: torch.Tensor | None = None
         self.sinks: torch.Tensor | None = None
         self.uk_t: torch.Tensor | None = None       # [heads, kv_rank, dim]: W_uk[h]^T, the key map moved to the query
         self.uv: torch.Tensor | None = None         # [heads, vdim, kv_rank]
+        self.ukv: torch.Tensor | None = None        # [heads * (dim + vdim), kv_rank]: both maps as they are, all keys' rows first
 
     def children(self) -> list[Part]:
         return [self.proj, self.o]
@@ -181,6 +186,9 @@ class RotaryLatentAttention(Mixer):
         self.sinks = get(f"{p}.sink").to(torch.float32).contiguous()
         self.uk_t = get(f"{p}.uk").view(self.heads, self.dim, self.kv_rank).transpose(1, 2).contiguous()
         self.uv = get(f"{p}.uv").view(self.heads, self.vdim, self.kv_rank).contiguous()
+        if self.rt.fast_kernels and self.expandable:
+            self.ukv = torch.cat([get(f"{p}.uk"), get(f"{p}.uv")], dim=0).contiguous()
+            self.uv = self.ukv[self.heads * self.dim:].view(self.heads, self.vdim, self.kv_rank)       # the same memory
 
     def cache_request(self) -> KVPages:
         return KVPages(1, self.key_size, 0, shared=True)
@@ -191,44 +199,101 @@ class RotaryLatentAttention(Mixer):
         return next(self.heads // s for s in range(1, self.heads + 1) if self.heads % s == 0 and self.heads // s <= TILE_ROWS)
 
     def plan_key(self) -> Optional[Hashable]:
-        return ("latent tiles", self.group) if self.rt.fast_kernels and self.scale > 0 else None
+        if not self.rt.fast_kernels or not self.scale > 0:
+            return None
+        return ("latent tiles", self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank)
 
     def plan(self, batch: BatchShape) -> Optional[StepPlan]:
-        """Tiles of up to 64 query rows; where single tokens are in the step, tiles of as few rows as one token needs (the
-        kernel's work follows the largest tile)."""
-        g = self.group
-        rows = -(-g // 16) * 16 if 1 in batch.q_lens else TILE_ROWS
-        tiles = tiles_of(batch.q_lens, g, rows)
-        return StepPlan({"all": np.asarray(tiles, dtype=np.int32).reshape(len(tiles), 4)}, {"rows": {"all": max(n for _, n, _, _ in tiles) * g}})
+        """"big": the portions whose keys and values are worth multiplying out (ops.latent_expansion_pays), in items of up to 256
+        tokens of the tensor-memory kernel, (first token, tokens, request, first row of the request), with "entries" (request,
+        first row, rows, 0).  "rest": the other tokens, in tiles of up to 64 query rows; where single tokens are among
+        them, of as few rows as one token needs (the kernel's work follows the largest tile).  The host's part says how many
+        rows there are in all and between which tokens the rest lies."""
+        key = (self.group, len(batch.q_lens)) if batch.max_q_len == 1 else None      # single tokens: the same tiles for every such step
+        if key in self._plans_of_single_tokens:
+            return self._plans_of_single_tokens[key]
+        g, T = self.group, sum(batch.q_lens)
+        spans = [batch.span_hint if batch.recorded else s + n for s, n in zip(batch.start_positions, batch.q_lens)]
+        row_bytes = 2 * self.heads * (self.dim + self.vdim)
+        entries, firsts, rows, t = [], {}, 0, 0
+        for i, (n, span) in enumerate(zip(batch.q_lens, spans)):
+            if (n >= BIG_PORTION and self.expandable and (rows + span) * row_bytes <= EXPANSION_BYTES
+                    and ops.latent_expansion_pays(n, span, self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank)):
+                entries.append((i, rows, span, 0))
+                firsts[i] = rows
+                rows += span
+        arrays, host = {}, {"rows": rows, "lo": 0, "hi": T}
+        if entries:
+            ids = set(firsts)
+            item = lambda n: [tl for tl in tiles_of(batch.q_lens, 1, n) if tl[2] in ids]
+            big = item(256)
+            if len(big) * self.heads < 148:                  # few items: half as long ones fill more SMs
+                big = item(128)
+            big.sort(key=lambda tl: -(batch.start_positions[tl[2]] + tl[3] + tl[1]))       # those that see the most keys first
+            arrays["big"] = np.asarray([(a, n, i, firsts[i]) for a, n, i, _ in big], dtype=np.int32)
+            arrays["entries"] = np.asarray(entries, dtype=np.int32)
+        rest = [n for i, n in enumerate(batch.q_lens) if i not in firsts]
+        if rest:
+            tile_rows = -(-g // 16) * 16 if 1 in rest else TILE_ROWS
+            tiles = [tl for tl in tiles_of(batch.q_lens, g, tile_rows) if tl[2] not in firsts]
+            arrays["rest"] = np.asarray(tiles, dtype=np.int32).reshape(len(tiles), 4)
+            host.update(tile_rows=max(n for _, n, _, _ in tiles) * g, lo=tiles[0][0], hi=tiles[-1][0] + tiles[-1][1])
+        plan = StepPlan(arrays, host)
+        if key is not None:
+            self._plans_of_single_tokens[key] = plan
+        return plan
 
-    def _attend(self, q_lat: torch.Tensor, mix: torch.Tensor, step: StepContext, cache: KVCacheView) -> None:
+    _plans_of_single_tokens: dict = {}
+
+    def _in_latent_space(self, gated: torch.Tensor, q: torch.Tensor, q_lat: torch.Tensor, gate: torch.Tensor, step: StepContext,
+                         cache: KVCacheView, plan, lo: int, hi: int) -> None:
+        """The tokens lo .. hi - 1 (others among them are overwritten later): the head's key map applied to the query, attention over
+        the cached vectors, the head's value map and gate."""
+        rt, L = self.rt, self.kv_rank
         table = step.block_tables[cache.group]
-        plan = step.plans.get(self.plan_key())
-        if plan is None or not ops.latent_flash_ok(self.key_size, self.kv_rank, self.group, cache.page_size):
+        ops.gemm_heads(q_lat[lo:hi, :, :L], q[lo:hi, :, :self.dim], self.uk_t, rt.stream)
+        mix = rt.empty((q.shape[0], self.heads, L))
+        if plan is None or not ops.latent_flash_ok(self.key_size, L, self.group, cache.page_size):
             ops.attention_plain(q_lat, mix, cache.k, cache.v, step.positions, step.token_seq, table, self.heads, 1, self.key_size,
-                                cache.page_size, 0, self.scale, self.rt.stream, v_dim=self.kv_rank, v_stride=self.key_size, sinks=self.sinks)
-            return
-        tiles = plan.arrays["all"]
-        splits = ops.latent_flash_splits(tiles.shape[0], self.heads // self.group, step.span_hint or step.max_context_len)
-        ops.latent_flash(q_lat, mix, cache.k, step.positions, table, tiles, plan.host["rows"]["all"], self.group, cache.page_size, self.scale,
-                         splits, self.rt.stream, sinks=self.sinks)
+                                cache.page_size, 0, self.scale, rt.stream, v_dim=L, v_stride=self.key_size, sinks=self.sinks)
+        else:
+            tiles = plan.arrays["rest"]
+            splits = ops.latent_flash_splits(tiles.shape[0], self.heads // self.group, step.span_hint or step.max_context_len)
+            ops.latent_flash(q_lat, mix, cache.k, step.positions, table, tiles, plan.host["tile_rows"], self.group, cache.page_size, self.scale,
+                             splits, rt.stream, sinks=self.sinks)
+        ops.gemm_heads(gated[lo:hi], mix[lo:hi], self.uv, rt.stream, gate=gate[lo:hi])
+
+    def _multiplied_out(self, gated: torch.Tensor, q: torch.Tensor, gate: torch.Tensor, step: StepContext, cache: KVCacheView, plan) -> None:
+        """The portions whose keys and values are formed for every head first."""
+        rt, rows = self.rt, plan.host["rows"]
+        lat = rt.empty((rows, self.key_size))
+        ops.latent_gather(lat, cache.k, plan.arrays["entries"], step.context_lens, step.block_tables[cache.group], cache.page_size, rt.stream)
+        kv = rt.empty((rows, self.heads * (self.dim + self.vdim)))
+        ops.linear(kv, lat[:, :self.kv_rank], self.ukv, rt.stream, fast=True)
+        tiles = plan.arrays["big"]
+        splits = ops.attention_tcgen05_splits(tiles.shape[0], self.heads, step.span_hint or step.max_context_len)
+        ops.latent_prefill(q, gated, kv, lat, step.positions, tiles, self.dim, self.rot_dim, self.kv_rank, self.scale, rt.stream, sinks=self.sinks,
+                           gate=gate, key_splits=splits)
 
     def forward(self, u: torch.Tensor, step: StepContext, cache: KVCacheView, write_cache: bool = True) -> torch.Tensor:
         rt = self.rt
-        T, H, L = u.shape[0], self.heads, self.kv_rank
+        T, H = u.shape[0], self.heads
         if not write_cache:
             raise ops.KernelError("latent attention always writes its own latents")
         n_q = H * (self.dim + self.rot_dim)
         pre = self.proj.forward(u, out_dtype=torch.float32)                  # q | dkv | g
         gate = pre[:, n_q + self.key_size:]
+        plan = step.plans.get(self.plan_key())
+        big = plan is not None and "big" in plan.arrays
+        rest = plan is None or "rest" in plan.arrays
         inv_freq, rot = self.position_encoding.rotary_table() if self.position_encoding is not None else (None, 0)
-        q, q_lat = rt.empty((T, H, self.dim + self.rot_dim)), rt.empty((T, H, self.key_size))
-        ops.latent_rope(pre, 0, n_q, H, self.dim, self.rot_dim, L, self.kv_norm_w, inv_freq, rot,
+        q, q_lat = rt.empty((T, H, self.dim + self.rot_dim)), rt.empty((T, H, self.key_size)) if rest else None
+        ops.latent_rope(pre, 0, n_q, H, self.dim, self.rot_dim, self.kv_rank, self.kv_norm_w, inv_freq, rot,
                         getattr(self.position_encoding, "magnitude", 1.0), q, q_lat, cache.k, step, step.block_tables[cache.group],
                         cache.page_size, self.eps, rt.stream)
         gated = rt.empty((T, H, self.vdim))
-        ops.gemm_heads(q_lat[:, :, :L], q[:, :, :self.dim], self.uk_t, rt.stream)       # the head's key map, applied to the query
-        mix = rt.empty((T, H, L))
-        self._attend(q_lat, mix, step, cache)
-        ops.gemm_heads(gated, mix, self.uv, rt.stream, gate=gate)
+        if rest:
+            self._in_latent_space(gated, q, q_lat, gate, step, cache, plan, plan.host["lo"] if plan else 0, plan.host["hi"] if plan else T)
+        if big:
+            self._multiplied_out(gated, q, gate, step, cache, plan)
         return self.o.forward(gated.view(T, H * self.vdim), out_dtype=self.out_dtype)

@@ -325,6 +325,74 @@ def test_many_heads_on_one_cached_vector(dtype, heads, dk, dv, page):
     assert ops.device_error() == 0
 
 
+@pytest.mark.parametrize("dk,page", [(48, 8), (576, 16), (8, 32)])
+def test_cached_vectors_are_gathered_row_by_row(dk, page):
+    from lucciola_b200 import ops
+    lens, starts = [3, 20, 1, 40], [0, 60, 9, 0]
+    step, _, pool, table, _ = latent_case(lens, starts, 1, dk, dk, page, torch.bfloat16, dk)
+    entries, first = [], 0
+    for i, rows in ((1, 128), (3, 40), (0, 7)):
+        entries.append((i, first, rows, 0))
+        first += rows
+    out = torch.full((first, dk), float("nan"), dtype=torch.bfloat16, device=DEV)
+    ops.latent_gather(out, pool, torch.tensor(entries, dtype=torch.int32, device=DEV), step.context_lens, table, page, stream())
+    for i, at, rows, _ in entries:
+        n = starts[i] + lens[i]
+        pos = torch.arange(n, device=DEV)
+        assert torch.equal(out[at:at + n], pool[table[i, pos // page].long(), 0, pos % page]) and not out[at + n:at + rows].any()
+
+
+@pytest.mark.parametrize("heads,dim,rot,vdim,rank", [(8, 128, 64, 128, 512), (3, 64, 32, 64, 192), (4, 32, 16, 64, 64), (5, 8, 8, 8, 40), (2, 40, 24, 104, 88), (2, 128, 0, 72, 64), (1, 72, 64, 128, 24)])
+def test_portions_on_multiplied_out_keys_and_values(heads, dim, rot, vdim, rank):
+    """Several portions of one batch, from the sequence's start and from further on, in items of one and two tiles and over key
+    ranges; a standing-out key at a block's edge, far back, at the query's own place and just behind it (where it must not be
+    seen); sinks and gates; rows behind a request's last one hold what would show."""
+    from lucciola_b200 import ops
+    from lucciola_b200.parts.attention import tiles_of
+    scale = 1.5 / (dim + rot) ** 0.5
+    g = torch.Generator(device=DEV).manual_seed(heads * dim)
+    r = lambda *s: torch.randn(*s, device=DEV, generator=g).to(torch.bfloat16)
+    for lens, starts, spot in (([300], [0], 63), ([17, 129], [200, 0], 64), ([256, 40], [128, 500], 0), ([128], [900], 899), ([33], [31], 10 ** 6)):
+        step = batch_of(lens, starts)
+        T = sum(lens)
+        firsts, rows = [], 0
+        for s, n in zip(starts, lens):
+            firsts.append(rows)
+            rows += s + n + 5                                              # five rows behind each request's last
+        q, kv, lat = r(T, heads, dim + rot), r(rows, heads * (dim + vdim)), r(rows, rank + rot)
+        t = 0
+        for f, s, n in zip(firsts, starts, lens):
+            last = q[t + n - 1, 0]
+            for at in ({min(spot, s + n - 1), s + n} if spot < 10 ** 6 else {s + n}):       # s + n: behind the last, not visible
+                kv[f + at, :dim] = 4.0 * last[:dim]
+                lat[f + at, rank:] = 4.0 * last[dim:]
+            t += n
+        pre = torch.randn(T, heads + 3, device=DEV, generator=g)
+        for sinks, gate in ((None, None), (torch.randn(heads, device=DEV, generator=g) * 3, pre[:, 3:]), (torch.full((heads,), 50.0, device=DEV), None)):
+            want = torch.zeros(T, heads, vdim, dtype=torch.float64, device=DEV)
+            t = 0
+            for f, s, n in zip(firsts, starts, lens):
+                K = torch.cat([kv[f:f + s + n, :heads * dim].reshape(s + n, heads, dim), lat[f:f + s + n, None, rank:].expand(-1, heads, -1)], dim=-1).double()
+                V = kv[f:f + s + n, heads * dim:].reshape(s + n, heads, vdim).double()
+                sc = torch.einsum("thd,jhd->htj", q[t:t + n].double(), K) * scale
+                j, i = torch.arange(s + n, device=DEV)[None], torch.arange(s, s + n, device=DEV)[:, None]
+                sc = sc.masked_fill(j > i, float("-inf"))
+                if sinks is not None:
+                    sc = torch.cat([sc, sinks.double()[:, None, None].expand(heads, n, 1)], dim=-1)
+                want[t:t + n] = torch.einsum("htj,jhd->thd", torch.softmax(sc, dim=-1)[..., :s + n], V)
+                t += n
+            if gate is not None:
+                want = want * torch.sigmoid(gate.double())[:, :, None]
+            for size in (256, 128):
+                tiles = torch.tensor([(a, n, 0, firsts[i]) for a, n, i, _ in tiles_of(lens, 1, size)], dtype=torch.int32, device=DEV)
+                for splits in (1, 2, 5):
+                    out = torch.full((T, heads, vdim), float("nan"), dtype=torch.bfloat16, device=DEV)
+                    ops.latent_prefill(q, out, kv, lat, step.positions, tiles, dim, rot, rank, scale, stream(), sinks=sinks, gate=gate, key_splits=splits)
+                    err = (out.double() - want).abs().max().item()
+                    assert err <= 1.5e-2 * max(want.abs().max().item(), 0.3), (lens, starts, size, splits, err)
+    assert ops.device_error() == 0
+
+
 def test_padding_entries_of_a_recorded_step_read_nothing():
     """An entry that owns no page beside one that does: finite output for it, whatever page 0 holds."""
     from lucciola_b200 import ops
@@ -341,9 +409,12 @@ def test_padding_entries_of_a_recorded_step_read_nothing():
 
 
 @pytest.mark.parametrize("dtype", TYPES)
+@pytest.mark.parametrize("way", ["as it comes", "multiplied out", "in latent space"])
 @pytest.mark.parametrize("layer", [("C", 0), ("C", 1), ("C", 2), ("C", 3), ("C", 4), ("A", 0), ("A", 1), ("D", 0), ("D", 1)])
-def test_a_mixer_alone(dtype, layer):
-    """Both kinds of mixer by themselves: a batch of unequal sequences that start at position 0, then one more token each."""
+def test_a_mixer_alone(dtype, layer, way, monkeypatch):
+    """Both kinds of mixer by themselves: a batch of unequal sequences that start at position 0, then one more token each, then
+    portions behind that; latent attention also with one of its two ways forced on every portion."""
+    from lucciola_b200 import ops
     from lucciola_b200.parts.base import BatchShape, KVCacheView, PlanView
     from lucciola_b200.config.registry import resolve_architecture
     name, i = layer
@@ -355,14 +426,18 @@ def test_a_mixer_alone(dtype, layer):
     part = model.blocks[i].mixer
     part.bind_all(lambda n: w[n].to(dtype).to(DEV))
     kind, m = cfg["layers"][i]["type"], cfg["layers"][i]["mixer"]
+    if way != "as it comes":
+        if kind != "latent_attention" or dtype == torch.float32:
+            pytest.skip("one way only")
+        monkeypatch.setattr(ops, "latent_expansion_pays", lambda *a: way == "multiplied out")
     sub = {k[len(f"l{i}.mix."):]: v.double() for k, v in w.items() if k.startswith(f"l{i}.mix.")}
     req, page = part.cache_request(), 16
-    lens, n_pages = [40, 3, 1, 130], 24
-    k_pool, table = scattered(n_pages, page, (req.num_kv_heads, req.head_dim), [n + 1 for n in lens], [0] * 4, dtype)
+    lens, more, n_pages = [40, 3, 1, 130], [17, 2, 150, 16], 40
+    k_pool, table = scattered(n_pages, page, (req.num_kv_heads, req.head_dim), [n + 1 + k for n, k in zip(lens, more)], [0] * 4, dtype)
     v_pool = k_pool if req.shared else torch.full((n_pages, req.num_kv_heads, page, req.v_head_dim or req.head_dim), float("nan"), dtype=dtype, device=DEV)
     cache, past = KVCacheView(k_pool, v_pool, 0, page), [None] * len(lens)
     W = cfg["width"]
-    for q_lens, starts in ((lens, [0] * 4), ([1] * 4, lens)):
+    for q_lens, starts in ((lens, [0] * 4), ([1] * 4, lens), (more, [n + 1 for n in lens])):
         step = batch_of(q_lens, starts)
         step.block_tables = [table]
         if part.plan_key() is not None:
