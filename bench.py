@@ -39,6 +39,9 @@ whose values are its keys, with a sink; a relu-squared feed-forward), beside Nel
 `--design nulalorn` does the same for the Nulalorn design (a norm in front of and behind every sublayer; two layers that run twice,
 each pass entered through a map of the stream and the embedding; window attention with capped scores on unit heads; gelu
 feed-forwards and experts named by a table of the token ids in turn), beside Bonolorn and Qwen3 at equal sizes.
+`--design kifezen` does the same for the Kifezen design (four residual streams with hyper-connections; latent attention with a
+rotated part and sinks in three of four layers, attention on unit heads with a query temperature in the fourth; gated
+feed-forwards and routed experts in turn), beside Riruzen, Nulalorn and Qwen3 at equal sizes.
 
 Peaks come from MEASURED_PEAKS.json beside this file when the driver wrote it, else from the
 fallback figures 6650 GB/s and 1590 TFLOP/s.  The timed work reads far more than the 126 MB of L2
@@ -447,7 +450,8 @@ DESIGN_SIZES = {
 
 # the models a --design run measures: the design and the nearest ones beside it
 DESIGN_BESIDE = {"riruzen": ("riruzen", "qwen3"), "bonolorn": ("riruzen", "qwen3", "bonolorn"), "nelovik": ("nelovik", "bonolorn", "qwen3"),
-                 "venitar": ("venitar", "nelovik", "qwen3"), "nulalorn": ("nulalorn", "bonolorn", "qwen3")}
+                 "venitar": ("venitar", "nelovik", "qwen3"), "nulalorn": ("nulalorn", "bonolorn", "qwen3"),
+                 "kifezen": ("kifezen", "riruzen", "nulalorn", "qwen3")}
 
 
 def design_configs(size: dict, layers: int, positions: int) -> dict:
@@ -512,7 +516,49 @@ def design_configs(size: dict, layers: int, positions: int) -> dict:
                 "layers": [{"type": "attention", "mixer": nmix, "mlp": ffd if i % 2 == 0 else nmoe} for i in range(layers - 2 if looped else layers)]}
     if looped:
         nulalorn["loop"] = {"start": 1, "stop": 3, "times": 2} if layers > 4 else {"start": 0, "stop": 2, "times": 2}
-    return {"riruzen": riruzen, "qwen3": qwen3, "bonolorn": bonolorn, "nelovik": nelovik, "venitar": venitar, "nulalorn": nulalorn}
+    # Kifezen: four streams; of every four layers three are latent attention (all heads of 128 + 64 rotated entries on a latent of
+    # 512, YaRN) and the third is attention on unit heads (a quarter as many kv heads, a temperature that steps every 512
+    # positions); layers take a gated feed-forward of the size's `ff` and 16 experts of `ff / 8` (4 a token) in turn
+    lat = {"heads": H, "dim": D, "rot_dim": 64, "vdim": D, "kv_rank": 512, "scale": (D + 64) ** -0.5,
+           "rot": {"dims": 64, "base": 1e4, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    unit = {"heads": H, "kv_heads": max(H // 4, 1), "dim": D, "vdim": D, "scale": D ** -0.5, "q_temp": {"coef": 0.1, "every": 512}}
+    kmoe = {"kind": "moe", "router": {"experts": 16, "top": 4}, "expert": {"ff": size["ff"] // 8}}
+    kifezen = {"architecture": "Kifezen", "vocab": size["vocab"], "width": W, "streams": 4, "norm": {"eps": 1e-6},
+               "layers": [{"type": "attention" if i % 4 == 2 else "latent_attention", "mixer": unit if i % 4 == 2 else lat,
+                           "mlp": ffd if i % 2 == 0 else kmoe} for i in range(layers)]}
+    return {"riruzen": riruzen, "qwen3": qwen3, "bonolorn": bonolorn, "nelovik": nelovik, "venitar": venitar, "nulalorn": nulalorn,
+            "kifezen": kifezen}
+
+
+def kifezen_costs(cfg: dict) -> dict:
+    """The same for a Kifezen configuration.  Latent layers count their maps from the latent to keys and values among the weights (a
+    prompt multiplies every position's out, a decoded token applies them to its query and to what it has gathered); attention
+    counts the heads' own sizes for a prompt.  Of the experts a step of B tokens reads at most B * top a layer (`expert_layers`)."""
+    W = cfg["width"]
+    weights = active = token_bytes = 0
+    attn, expert_layers = [], []
+    for l in cfg["layers"]:
+        m, f = l["mixer"], l["mlp"]
+        H, D, Vd = m["heads"], m["dim"], m["vdim"]
+        weights += H * W + W * H * Vd
+        if l["type"] == "attention":
+            weights += (H * D + m["kv_heads"] * (D + Vd)) * W
+            token_bytes += 2 * m["kv_heads"] * (D + Vd)
+            attn.append(lambda T, H=H, D=D, Vd=Vd: H * 2.0 * (D + Vd) * (T * (T + 1) / 2))
+        else:
+            R, L = m["rot_dim"], m["kv_rank"]
+            weights += (H * (D + R) + L + R) * W + H * (D + Vd) * L
+            token_bytes += 2 * (L + R)
+            attn.append(lambda T, H=H, D=D, R=R, Vd=Vd: H * 2.0 * (D + R + Vd) * (T * (T + 1) / 2))
+        if f["kind"] == "dense":
+            weights += 3 * f["ff"] * W
+        else:
+            one = 3 * f["expert"]["ff"] * W
+            weights += f["router"]["experts"] * W
+            expert_layers.append((one, f["router"]["experts"], f["router"]["top"]))
+            active += f["router"]["top"] * one
+    return {"weight_bytes": 2 * (weights + cfg["vocab"] * W), "token_bytes": token_bytes, "request_bytes": 0, "flops_per_token": 2.0 * (weights + active),
+            "attn_flops": lambda T: sum(f(T) for f in attn), "expert_layers": expert_layers}
 
 
 def nulalorn_costs(cfg: dict) -> dict:
@@ -649,6 +695,8 @@ def design_costs(name: str, cfg: dict) -> dict:
         return venitar_costs(cfg)
     if name == "nulalorn":
         return nulalorn_costs(cfg)
+    if name == "kifezen":
+        return kifezen_costs(cfg)
     if name == "qwen3":
         L = cfg["num_hidden_layers"]
         per_layer, weight_bytes, kv = model_bytes_and_flops(cfg, L)
@@ -707,7 +755,7 @@ def run_design(args) -> int:
             pages = 64 * (-(-(ctx + K + Wm + 8) // page)) + -(-T // page) + 64
             options = EngineOptions(dtype="bfloat16", block_size=page, max_blocks=pages, max_num_seqs=66, max_tokens_per_step=T + 64,
                                     use_cuda_graph=not (args.no_graph or args.profile))
-            if args.design in ("venitar", "nulalorn"):
+            if args.design in ("venitar", "nulalorn", "kifezen"):
                 # designs whose positions have no limit of their own get the run's: block tables as wide as the run needs
                 options = EngineOptions(dtype="bfloat16", block_size=page, max_blocks=pages, max_num_seqs=66, max_tokens_per_step=T + 64,
                                         use_cuda_graph=not (args.no_graph or args.profile), max_model_len=max(ctx, T) + K + Wm + 64)
@@ -814,12 +862,12 @@ def main() -> int:
     ap.add_argument("--portion", type=int, default=512, help="tokens of the portion of a --profile mixed step")
     ap.add_argument("--time-kernel", choices=["attention_key_ranges"], default=None,
                     help="time one kernel alone over a grid of sizes, print a line of JSON a case, and exit")
-    ap.add_argument("--design", choices=["riruzen", "bonolorn", "nelovik", "venitar", "nulalorn"], default=None,
+    ap.add_argument("--design", choices=["riruzen", "bonolorn", "nelovik", "venitar", "nulalorn", "kifezen"], default=None,
                     help="instead of the default workload: prefill and decode of this design beside the Qwen3 decoder at equal "
                          "sizes (--design-sizes; --layers, default 8; --prefill-tokens; --context up to 2048; --profile decode|prefill "
                          "with --batch runs one step between cudaProfilerStart/Stop)")
     ap.add_argument("--design-sizes", default="w2048,w4096", help="which of %s" % ", ".join(sorted(DESIGN_SIZES)))
-    ap.add_argument("--design-models", default="", help="which of riruzen, qwen3, bonolorn, nelovik, venitar, nulalorn (empty: the design and those beside it)")
+    ap.add_argument("--design-models", default="", help="which of riruzen, qwen3, bonolorn, nelovik, venitar, nulalorn, kifezen (empty: the design and those beside it)")
     args = ap.parse_args()
     if args.time_kernel == "attention_key_ranges":
         return time_attention_key_ranges()

@@ -452,44 +452,71 @@ __global__ void __launch_bounds__(256) expert_gemm_mma_kernel(ExpertGemmParams p
       }
 }
 
-// The same without a gate for steps with a few pairs an expert, on row tiles of at most 16 places (the dispatch is told so): the
-// launch is a stream of weights, so nearly all shared memory holds stages of weights, six of them in flight.  A CTA of four
-// warps takes 64 output columns, a warp 16.  Sums in the order of the kernel above.
-constexpr int EF_BM = 16, EF_BN = 64, EF_BK = 64, EF_LD = EF_BK + 8, EF_STAGES = 6;
-constexpr int EF_SMEM = EF_STAGES * (EF_BM + EF_BN) * EF_LD * 2;
+// The same for steps with a few pairs an expert: the launch is a stream of weights, so nearly all shared memory holds stages of
+// weights, six of them in flight.  Row tiles of at most 16 MT places (the dispatch is told so; row blocks of 16 that hold no place
+// are neither fetched nor multiplied).  A CTA of four warps takes 64 rows of weights, a warp 16: 64 output columns, or, gated, the
+// gate and the up rows of 32, the eight of a warp side by side so that both sums of a column meet in one thread.  Sums in the
+// order of the kernel above.
+constexpr int EF_BN = 64, EF_BK = 64, EF_LD = EF_BK + 8, EF_STAGES = 6;
+template <int MT>
+constexpr int expert_few_smem() { return EF_STAGES * (16 * MT + EF_BN) * EF_LD * 2; }
 
-template <typename TY>
+template <typename TY, bool GATED, int MT>
 __global__ void __launch_bounds__(128) expert_gemm_few_kernel(ExpertGemmParams p) {
+  constexpr int BM = 16 * MT;
   extern __shared__ __align__(16) uint8_t ex_smem[];
   bf16* As = reinterpret_cast<bf16*>(ex_smem);                    // [stage][BM][LD]
-  bf16* Bs = As + EF_STAGES * EF_BM * EF_LD;                      // [stage][BN][LD]
+  bf16* Bs = As + EF_STAGES * BM * EF_LD;                         // [stage][BN][LD]
   pdl_trigger();
   pdl_wait();
   if ((int)blockIdx.y >= p.meta[0]) return;
   const int* m = p.meta + 4 + 3 * blockIdx.y;
-  const int e = m[0], r0 = m[1], r1 = min(m[2], m[1] + EF_BM);
+  const int e = m[0], r0 = m[1], r1 = min(m[2], m[1] + BM);
+  const int blocks = (r1 - r0 + 15) >> 4;                         // row blocks that hold places
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int n0 = blockIdx.x * EF_BN, wn = warp * 16;
+  const int ncols = GATED ? p.N / 2 : p.N;
+  const int n0 = blockIdx.x * (GATED ? EF_BN / 2 : EF_BN), wn = warp * 16;
   const bf16* x = (const bf16*)p.x;
   const bf16* w = (const bf16*)p.w + (size_t)e * p.N * p.K;
-  const int c_r = tid >> 3, c_c = (tid & 7) * 8;                  // this thread's row of A, and of every 16 rows of B; its 16-byte piece
-  const int place = r0 + c_r;
-  const int a_row = place < r1 ? (p.gather ? p.pair_at[place] / p.top : place) : -1;
+  const int c_r = tid >> 3, c_c = (tid & 7) * 8;                  // this thread's row of every 16 rows of A and of B; its 16-byte piece
+  int a_row[MT];
+#pragma unroll
+  for (int i = 0; i < MT; ++i) {
+    const int place = r0 + c_r + 16 * i;
+    a_row[i] = place < r1 ? (p.gather ? p.pair_at[place] / p.top : place) : -1;
+  }
+  const bf16* w_row[EF_BN / 16];                                  // null: past the last column
+#pragma unroll
+  for (int it = 0; it < EF_BN / 16; ++it) {
+    const int r = c_r + it * 16;
+    if (GATED) {
+      const int n = n0 + (r >> 4) * 8 + (r & 7);
+      int gr, ur;
+      gate_up_rows(p, n, ncols, gr, ur);
+      w_row[it] = n < ncols ? w + (size_t)((r >> 3) & 1 ? ur : gr) * p.K + c_c : nullptr;
+    } else {
+      w_row[it] = n0 + r < p.N ? w + (size_t)(n0 + r) * p.K + c_c : nullptr;
+    }
+  }
   auto load_stage = [&](int st, int k0) {
     const bool k_ok = k0 + c_c < p.K;
-    ex_cp_async16(As + (st * EF_BM + c_r) * EF_LD + c_c, a_row >= 0 && k_ok ? x + (size_t)a_row * p.ldx + k0 + c_c : x, a_row >= 0 && k_ok);
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+      if (i < blocks)
+        ex_cp_async16(As + (st * BM + c_r + 16 * i) * EF_LD + c_c, a_row[i] >= 0 && k_ok ? x + (size_t)a_row[i] * p.ldx + k0 + c_c : x, a_row[i] >= 0 && k_ok);
 #pragma unroll
     for (int it = 0; it < EF_BN / 16; ++it) {
-      const int r = c_r + it * 16;
-      const bool ok = k_ok && n0 + r < p.N;
-      ex_cp_async16(Bs + (st * EF_BN + r) * EF_LD + c_c, ok ? w + (size_t)(n0 + r) * p.K + k0 + c_c : w, ok);
+      const bool ok = k_ok && w_row[it] != nullptr;
+      ex_cp_async16(Bs + (st * EF_BN + c_r + it * 16) * EF_LD + c_c, ok ? w_row[it] + k0 : w, ok);
     }
   };
-  float acc[2][4];
+  float acc[MT][2][4];
 #pragma unroll
-  for (int j = 0; j < 2; ++j)
+  for (int i = 0; i < MT; ++i)
 #pragma unroll
-    for (int k = 0; k < 4; ++k) acc[j][k] = 0.f;
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) acc[i][j][k] = 0.f;
   const int nk = (p.K + EF_BK - 1) / EF_BK;
 #pragma unroll
   for (int st = 0; st < EF_STAGES - 1; ++st) {
@@ -506,27 +533,51 @@ __global__ void __launch_bounds__(128) expert_gemm_few_kernel(ExpertGemmParams p
     asm volatile("cp.async.commit_group;" ::: "memory");
 #pragma unroll
     for (int kk = 0; kk < EF_BK; kk += 16) {
-      uint32_t a[4], b0, b1, b2, b3;
-      ex_ldmatrix_x4(As + (st * EF_BM + a_lr) * EF_LD + kk + a_lk, a[0], a[1], a[2], a[3]);
+      uint32_t b0, b1, b2, b3;
       ex_ldmatrix_x4(Bs + (st * EF_BN + wn + b_lr) * EF_LD + kk + b_lk, b0, b1, b2, b3);
       const uint32_t lo[2] = {b0, b1}, hi[2] = {b2, b3};
-      ex_mma_16816(acc[0], a, lo);
-      ex_mma_16816(acc[1], a, hi);
+#pragma unroll
+      for (int i = 0; i < MT; ++i)
+        if (i < blocks) {
+          uint32_t a[4];
+          ex_ldmatrix_x4(As + (st * BM + 16 * i + a_lr) * EF_LD + kk + a_lk, a[0], a[1], a[2], a[3]);
+          ex_mma_16816(acc[i][0], a, lo);
+          ex_mma_16816(acc[i][1], a, hi);
+        }
     }
   }
   TY* y = (TY*)p.y;
 #pragma unroll
-  for (int nb = 0; nb < 2; ++nb)
+  for (int i = 0; i < MT; ++i)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int row = r0 + (lane >> 2) + 8 * half;
+      const int row = r0 + 16 * i + (lane >> 2) + 8 * half;
       if (row >= r1) continue;
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
-        const int n = n0 + wn + nb * 8 + 2 * (lane & 3) + j;
-        if (n < p.N) y[(size_t)row * p.ldy + n] = from_f32<TY>(post_op(p.post, 0.f, acc[nb][2 * half + j]));
+        if (GATED) {
+          const int n = n0 + warp * 8 + 2 * (lane & 3) + j;
+          if (n < ncols) y[(size_t)row * p.ldy + n] = from_f32<TY>(expert_act(p.act, p.limit, acc[i][0][2 * half + j], acc[i][1][2 * half + j]));
+        } else {
+#pragma unroll
+          for (int nb = 0; nb < 2; ++nb) {
+            const int n = n0 + wn + nb * 8 + 2 * (lane & 3) + j;
+            if (n < p.N) y[(size_t)row * p.ldy + n] = from_f32<TY>(post_op(p.post, 0.f, acc[i][nb][2 * half + j]));
+          }
+        }
       }
     }
+}
+
+template <typename TY, bool GATED, int MT>
+void launch_expert_few(const ExpertGemmParams& p, int ncols, int max_tiles, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    cudaFuncSetAttribute(expert_gemm_few_kernel<TY, GATED, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, expert_few_smem<MT>());
+    configured = true;
+  }
+  const int cols = GATED ? EF_BN / 2 : EF_BN;
+  launch(expert_gemm_few_kernel<TY, GATED, MT>, dim3((ncols + cols - 1) / cols, max_tiles), dim3(128), expert_few_smem<MT>(), stream, p);
 }
 
 // ---- combine ---------------------------------------------------------------------------------------------------
@@ -575,15 +626,16 @@ LB_EXPORT int lb_route_topk(int* ids, float* weights, const float* logits, long 
   return 0;
 }
 
-// The row tiles of the experts' products have this many places; those of steps with a few pairs an expert `few` of them.
-LB_EXPORT int lb_expert_tile_rows(int few) { return few ? lb::EF_BM : lb::EX_BM; }
+// The places of a row tile of the experts' products; few: 1 for steps with a few pairs an expert (tiles of 16 places), 2 for those
+// with some more (the same kernel, tiles of 64).
+LB_EXPORT int lb_expert_tile_rows(int few) { return few == 1 ? 16 : lb::EX_BM; }
 
 // ids [pairs] -> offsets [experts + 1], pair_at [pairs], place_of [pairs], meta [4 + 3 * (pairs / tile_rows + experts)]
 // (tokens != null: ids is the table [vocab, top] and pairs = tokens * top; its entries lie in 0 .. experts - 1)
 // tile_rows: lb_expert_tile_rows of the product that will walk the tiles
 LB_EXPORT int lb_expert_dispatch(const int* ids, const int* tokens, int top, int pairs, int experts, int tile_rows, int* offsets, int* pair_at,
                                  int* place_of, int* meta, cudaStream_t stream) {
-  LB_CHECK_ARG(tile_rows == lb::EX_BM || tile_rows == lb::EF_BM, "expert_dispatch: row tiles of %d places", tile_rows);
+  LB_CHECK_ARG(tile_rows == lb::EX_BM || tile_rows == 16, "expert_dispatch: row tiles of %d places", tile_rows);
   LB_CHECK_ARG(tokens == nullptr || (top > 0 && pairs % top == 0), "expert_dispatch: %d pairs are not %d choices a token", pairs, top);
   LB_CHECK_ARG(ids && offsets && pair_at && place_of && meta, "expert_dispatch: null argument");
   LB_CHECK_ARG(pairs >= 0 && experts > 0 && experts <= 4096, "expert_dispatch: bad sizes pairs=%d experts=%d", pairs, experts);
@@ -635,16 +687,17 @@ LB_EXPORT int lb_expert_gemm(void* y, int y_dtype, const void* x, int x_dtype, c
   p.gather = gather; p.gated = gated; p.act = act; p.limit = limit; p.interleaved = interleaved; p.post = post;
   const int ncols = gated ? N / 2 : N;
   const bool mma = fast && x_dtype == LB_BF16 && w_dtype == LB_BF16 && K % 8 == 0 && ldx % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0;
-  LB_CHECK_ARG(!few || (mma && !gated), "expert_gemm: tiles of a few places are for ungated bfloat16 products on the tensor cores");
+  LB_CHECK_ARG(few >= 0 && few <= 2 && (!few || mma), "expert_gemm: the kernel for few pairs an expert is for bfloat16 products on the tensor cores");
   if (few) {
-    static bool few_set = false;
-    if (!few_set) {
-      cudaFuncSetAttribute(lb::expert_gemm_few_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::EF_SMEM);
-      cudaFuncSetAttribute(lb::expert_gemm_few_kernel<lb::bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, lb::EF_SMEM);
-      few_set = true;
-    }
-    dim3 grid((N + lb::EF_BN - 1) / lb::EF_BN, max_tiles);
-    LB_DISPATCH_DTYPE(y_dtype, TY, { lb::launch(lb::expert_gemm_few_kernel<TY>, grid, dim3(128), lb::EF_SMEM, stream, p); })
+    LB_DISPATCH_DTYPE(y_dtype, TY, {
+      if (gated) {
+        if (few == 1) lb::launch_expert_few<TY, true, 1>(p, ncols, max_tiles, stream);
+        else lb::launch_expert_few<TY, true, 4>(p, ncols, max_tiles, stream);
+      } else {
+        if (few == 1) lb::launch_expert_few<TY, false, 1>(p, ncols, max_tiles, stream);
+        else lb::launch_expert_few<TY, false, 4>(p, ncols, max_tiles, stream);
+      }
+    })
   } else if (mma) {
     static bool attr_set = false;
     if (!attr_set) {       // the stages need more shared memory than a launch gets unasked

@@ -350,6 +350,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
 constexpr int LF_MAX_SPLITS = 64;
 __global__ void __launch_bounds__(128) latent_flash_combine_kernel(LatentFlashParams p) {
   __shared__ float wz[LF_MAX_SPLITS];
+  __shared__ float den_s;
   pdl_trigger();
   const int4 tile = p.tiles[blockIdx.y];
   const int hg = blockIdx.z, r = blockIdx.x, G = p.group;
@@ -358,28 +359,38 @@ __global__ void __launch_bounds__(128) latent_flash_combine_kernel(LatentFlashPa
   const float sink = p.sinks ? p.sinks[head] * 1.4426950408889634f : -INFINITY;
   pdl_wait();
   const size_t base = ((size_t)blockIdx.y * gridDim.z + hg) * p.splits;
-  float M = sink;
-  for (int z = 0; z < p.splits; ++z) M = fmaxf(M, p.part_ml[((base + z) * p.part_rows + r) * 2]);
-  for (int z = threadIdx.x; z < p.splits; z += blockDim.x) {
-    const float mz = p.part_ml[((base + z) * p.part_rows + r) * 2];
-    wz[z] = mz == -INFINITY ? 0.f : exp2f(mz - M);
+  if (threadIdx.x < 32) {                      // the ranges' weights: a lane two of them
+    float2 ml[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int z = threadIdx.x + 32 * u;
+      ml[u] = z < p.splits ? *reinterpret_cast<const float2*>(p.part_ml + ((base + z) * p.part_rows + r) * 2) : make_float2(-INFINITY, 0.f);
+    }
+    const float M = fmaxf(sink, warp_max(fmaxf(ml[0].x, ml[1].x)));
+    float den = 0.f;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const float w = ml[u].x == -INFINITY ? 0.f : exp2f(ml[u].x - M);
+      wz[threadIdx.x + 32 * u] = w;
+      den += ml[u].y * w;
+    }
+    den = warp_sum(den) + (sink == -INFINITY ? 0.f : exp2f(sink - M));
+    if (threadIdx.x == 0) den_s = den;
   }
   __syncthreads();
-  float den = sink == -INFINITY ? 0.f : exp2f(sink - M);
-  for (int z = 0; z < p.splits; ++z) if (wz[z] != 0.f) den += p.part_ml[((base + z) * p.part_rows + r) * 2 + 1] * wz[z];
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  const float inv = den_s > 0.f ? 1.f / den_s : 0.f;
   bf16* dst = p.out + ((size_t)(tile.x + r / G) * p.heads + head) * p.dv;
   for (int e = threadIdx.x * 4; e < p.dv; e += blockDim.x * 4) {
     float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int z0 = 0; z0 < p.splits; z0 += 4) {
-      float4 a[4];
+    for (int z0 = 0; z0 < p.splits; z0 += 8) {
+      float4 a[8];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
+      for (int u = 0; u < 8; ++u) {
         const bool have = z0 + u < p.splits && wz[z0 + u] != 0.f;        // what weighs nothing may never have been written
         a[u] = have ? *reinterpret_cast<const float4*>(p.part_o + ((base + z0 + u) * p.part_rows + r) * p.dv + e) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
+      for (int u = 0; u < 8; ++u)
         if (z0 + u < p.splits) {
           const float w = wz[z0 + u];
           acc.x = fmaf(w, a[u].x, acc.x); acc.y = fmaf(w, a[u].y, acc.y); acc.z = fmaf(w, a[u].z, acc.z); acc.w = fmaf(w, a[u].w, acc.w);

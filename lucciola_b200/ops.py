@@ -1015,15 +1015,15 @@ def route_topk(ids: torch.Tensor, weights: torch.Tensor, logits: torch.Tensor, c
           T, E, ids.shape[1], groups, keep, scale, 1 if softmax else 0, stream)
 
 
-def expert_tile_rows(few: bool = False) -> int:
-    """Places of a row tile of the experts' products; `few`: of those for steps with a few pairs an expert."""
+def expert_tile_rows(few: int = 0) -> int:
+    """Places of a row tile of the experts' products; `few`: of those for steps with a few pairs an expert (1), or some more (2)."""
     lib = library()
     lib.lb_expert_tile_rows.argtypes = [c_int]
     lib.lb_expert_tile_rows.restype = c_int
-    return int(lib.lb_expert_tile_rows(1 if few else 0))
+    return int(lib.lb_expert_tile_rows(int(few)))
 
 
-def expert_max_tiles(pairs: int, experts: int, few: bool = False) -> int:
+def expert_max_tiles(pairs: int, experts: int, few: int = 0) -> int:
     """The most row tiles the experts' products can have for this many (token, choice) pairs."""
     return -(-pairs // expert_tile_rows(few)) + experts
 
@@ -1036,11 +1036,11 @@ def _dispatch_pairs(ids: torch.Tensor, tokens: torch.Tensor | None) -> tuple[int
 
 
 def expert_dispatch(ids: torch.Tensor, experts: int, offsets: torch.Tensor, pair_at: torch.Tensor, place_of: torch.Tensor,
-                    meta: torch.Tensor, stream: int, tokens: torch.Tensor | None = None, few: bool = False) -> None:
+                    meta: torch.Tensor, stream: int, tokens: torch.Tensor | None = None, few: int = 0) -> None:
     """Sort the (token, choice) pairs by expert, on the device: offsets [experts + 1], pair_at [pairs] (the pair at each
     place), place_of [pairs], meta [4 + 3 * expert_max_tiles] (the row tiles of the products).  ids: the experts of the pairs, [T, top], or, with the step's
     `tokens` [T], a table [vocab, top] whose row of a token's id holds the token's experts (entries in 0 .. experts - 1).
-    `few`: row tiles for expert_gemm(few=True)."""
+    `few`: row tiles for expert_gemm with the same `few`."""
     for t, what in ((ids, "expert ids"), (offsets, "offsets"), (pair_at, "pair list"), (place_of, "places"), (meta, "tile list")):
         _check(t, what, torch.int32)
     pairs, top = _dispatch_pairs(ids, tokens)
@@ -1052,12 +1052,12 @@ def expert_dispatch(ids: torch.Tensor, experts: int, offsets: torch.Tensor, pair
 
 def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.Tensor, pair_at: torch.Tensor, top: int,
                 gather: bool, stream: int, act: str | None = None, limit: float = 0.0, fast: bool = True,
-                interleaved: bool = False, post: str | None = None, few: bool = False) -> None:
+                interleaved: bool = False, post: str | None = None, few: int = 0) -> None:
     """y[place] = x[row(place)] . w[e]^T for the places of every expert e (see expert_dispatch); w [experts, N, K].
     `gather`: row(place) is the pair's token, else the place.  With `act`, w[e] is N/2 gate rows then N/2 up rows (or,
     `interleaved`, blocks of 64 gate rows and their 64 up rows in turn, see interleave_gate_up) and y[place] =
     act(gate) * up with N/2 columns.  `post` (without act): an element operation on the sums, see POST_OPS.
-    `few` (without act, bfloat16): row tiles of few places, see expert_dispatch; the weights then stream through a kernel of their own."""
+    `few` (bfloat16): 1, row tiles of 16 places, or 2, of 64 (see expert_dispatch): the weights stream through a kernel made for that."""
     _check(y, "expert output"); _check(x, "expert input"); _check(w, "expert weights")
     E, N, K = w.shape
     pairs = pair_at.numel()
@@ -1067,7 +1067,7 @@ def expert_gemm(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor, meta: torch.T
     _call("lb_expert_gemm", y.data_ptr(), dtype_code(y.dtype), x.data_ptr(), dtype_code(x.dtype), w.data_ptr(), dtype_code(w.dtype),
           meta.data_ptr(), pair_at.data_ptr(), expert_max_tiles(pairs, E, few), N, K, K, cols, top, 1 if gather else 0,
           1 if act is not None else 0, GATE_ACTS[act] if act is not None else 0, limit, 1 if fast else 0, 1 if interleaved else 0,
-          POST_OPS[post], 1 if few else 0, stream)
+          POST_OPS[post], int(few), stream)
 
 
 GROUP_TILE = 128          # token tile of the grouped tensor-memory product

@@ -40,9 +40,9 @@ from .linear import Linear
 # From this many pairs of token and choice an expert (on average) the padded runs of the tensor-memory product cost
 # less than they gain: the padding is 64 places an expert on average, 127 at most, and the product several times faster.
 GROUPED_FROM = 96
-# Up to this many pairs an expert (on average) an ungated step is a stream of the experts' weights and takes the kernel made for
-# it, whose row tiles have 16 places (an expert with more reads its weights once a tile).
-FEW_UP_TO = 8
+# Up to so many pairs an expert (on average) a step is a stream of the experts' weights and takes the kernel made for it, with row
+# tiles of 16 places (an expert with more reads its weights once a tile), or of 64 from FEW_UP_TO on.
+FEW_UP_TO, SOME_UP_TO = 8, 48
 
 
 @dataclass
@@ -52,7 +52,7 @@ class Dispatch:
     place_of: torch.Tensor
     meta: Optional[torch.Tensor] = None             # the row tiles of the runs; None: runs padded to whole tiles, then
     tile_group: Optional[torch.Tensor] = None       # the expert of each tile
-    few: bool = False                               # row tiles of few places
+    few: int = 0                                    # the kernel for few pairs an expert, see ops.expert_gemm
 
 
 class ExpertBank(FeedForward):
@@ -107,7 +107,7 @@ class ExpertBank(FeedForward):
             ops.expert_dispatch_padded(ids, E, pair_at, place_of, tile_group, rt.stream, tokens=tokens)
             return Dispatch(pair_at, place_of, tile_group=tile_group)
         offsets, pair_at = rt.empty((E + 1,), torch.int32), rt.empty((pairs,), torch.int32)
-        few = self.grouped_ok and not self.gated and pairs <= FEW_UP_TO * E
+        few = 0 if not self.grouped_ok else 1 if pairs <= FEW_UP_TO * E else 2 if pairs <= SOME_UP_TO * E else 0
         meta = rt.empty((4 + 3 * ops.expert_max_tiles(pairs, E, few),), torch.int32)
         ops.expert_dispatch(ids, E, offsets, pair_at, place_of, meta, rt.stream, tokens=tokens, few=few)
         return Dispatch(pair_at, place_of, meta=meta, few=few)

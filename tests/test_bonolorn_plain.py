@@ -148,7 +148,7 @@ def test_the_measurement_configurations_are_valid():
     from lucciola_b200.config import resolve_architecture
     for size in bench.DESIGN_SIZES.values():
         cfgs = bench.design_configs(size, 4, 4096)
-        assert set(cfgs) == {"bonolorn", "riruzen", "qwen3", "nelovik", "venitar", "nulalorn"}
+        assert set(cfgs) == {"bonolorn", "riruzen", "qwen3", "nelovik", "venitar", "nulalorn", "kifezen"}
         for name, cfg in cfgs.items():
             arch = resolve_architecture(cfg)
             arch.config_from_dict(cfg)

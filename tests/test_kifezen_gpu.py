@@ -211,7 +211,7 @@ def test_router_with_a_softmax_over_the_chosen(experts, top):
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("experts,top,width,ff,lens", [(5, 2, 70, 28, [3, 1, 9]), (1, 1, 40, 32, [1]), (16, 4, 256, 64, [1] * 8), (12, 1, 200, 72, [40]),
+@pytest.mark.parametrize("experts,top,width,ff,lens", [(5, 2, 70, 28, [3, 1, 9]), (1, 1, 40, 32, [1]), (16, 4, 256, 64, [1] * 8), (12, 1, 200, 72, [40]), (16, 4, 264, 64, [60]), (3, 2, 128, 128, [20, 9]),
                                                        (2, 2, 256, 64, [130, 70]), (6, 3, 128, 192, [400, 3])])
 def test_experts_weighted_by_a_softmax_over_the_chosen(dtype, experts, top, width, ff, lens):
     """The whole part with independent experts: short runs of tokens and runs long enough for the tensor-memory product
@@ -243,7 +243,7 @@ def test_experts_weighted_by_a_softmax_over_the_chosen(dtype, experts, top, widt
 
 
 @pytest.mark.parametrize("dtype", TYPES)
-@pytest.mark.parametrize("T,H,K,N", [(5, 3, 16, 24), (70, 8, 128, 512), (1, 2, 64, 40), (33, 4, 10, 14)])
+@pytest.mark.parametrize("T,H,K,N", [(5, 3, 16, 24), (70, 8, 128, 512), (1, 2, 64, 40), (33, 4, 10, 14), (8, 5, 512, 128), (64, 3, 512, 136), (20, 2, 200, 33), (64, 2, 1000, 40)])
 def test_per_head_products_on_parts_of_heads_with_a_gate_a_head(dtype, T, H, K, N):
     from lucciola_b200 import ops
     x, y = torch.randn(T, H, K + 8, device=DEV).to(dtype), torch.full((T, H, N + 16), float("nan"), device=DEV).to(dtype)
