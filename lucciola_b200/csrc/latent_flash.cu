@@ -7,8 +7,9 @@
 // query rows share every cached vector the CTA reads.  The keys of a tile may be cut into `splits` ranges (grid z) whose
 // unnormalised results (m, l, o) a second kernel adds up in the ranges' order.
 //
-// Per CTA a ninth warp fetches: stages of 64 cached vectors by TMA (boxes of 64 entries x the page's tokens, 128-byte
-// swizzle; what lies past dk reads as zeros).  The eight computing warps work on a stage in two phases:
+// Per CTA a ninth warp fetches: stages of 64 cached vectors by TMA, in groups of eight: one box brings all entries of a group's
+// vectors, as chunks of 64 entries x 8 vectors in the 128-byte swizzle (a CTA can issue a box in some hundred cycles
+// whatever its size, so few large ones; sizes that are no multiple of 64 take a box a chunk, which reads zeros past dk).  The eight computing warps work on a stage in two phases:
 //     S = Q K^T    the MT row blocks of 16 times the 64 keys are shared out (MT = 1: 8 keys a warp, 2: one row block and 16
 //                  keys, 4: one row block and 32 keys); maxima meet through shared memory; P goes there in bfloat16
 //     O += P V     each warp owns an eighth of the value entries for ALL rows, so the values are read once from shared
@@ -40,12 +41,18 @@ struct LatentFlashParams {
   int part_rows, splits;
   int heads, group, dk, dv, page_size, page_shift;
   float scale_log2;                           // scale * log2(e)
+  int whole;                                  // 1: a box brings whole vectors (dk a multiple of 64)
 };
 
 __device__ __forceinline__ void lf_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
-__device__ __forceinline__ void lf_tma_2d(uint32_t dst, const CUtensorMap* map, int x, int y, uint32_t bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
-               ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(bar) : "memory");
+__device__ __forceinline__ void lf_tma_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+               ::"r"(dst), "l"(map), "r"(x), "r"(y), "r"(z), "r"(bar) : "memory");
+}
+// Byte offset of 16-byte piece c (over the whole vector) of vector r in a stage: groups of eight vectors, chunks of 64 entries.
+template <int NK>
+__device__ __forceinline__ uint32_t lf_stage_offset(int r, int c) {
+  return (uint32_t)((r >> 3) * (NK * 1024) + (c >> 3) * 1024 + (r & 7) * 128 + (((c & 7) ^ (r & 7)) << 4));
 }
 // Byte offset of 16-byte piece c (over the whole row) of row r in a matrix of `rows` rows cut into chunks of 64 entries.
 __device__ __forceinline__ uint32_t lf_offset(int rows, int r, int c) {
@@ -106,18 +113,19 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
 
   if (warp == LF_WARPS) {
     // ---- the fetching warp ------------------------------------------------------------------------------------------------
-    const int box_keys = min(p.page_size, LF_KEYS);
-    const int boxes = LF_KEYS / box_keys;
+    const int pieces = p.whole ? 1 : NK;                       // boxes of a group of eight vectors
     auto fetch = [&](int st) {
       const int b = st % STAGES;
       if (lane == 0) mbar_expect_tx(full(b), STAGE_BYTES);
       __syncwarp();
-      for (int op = lane; op < boxes * NK; op += 32) {
-        const int box = op / NK, chunk = op % NK;
-        const int key0 = kbeg + st * LF_KEYS + box * box_keys;
+      for (int op = lane; op < 8 * pieces; op += 32) {
+        const int group = op / pieces, chunk = op - group * pieces;
+        const int key0 = kbeg + st * LF_KEYS + group * 8;
         const int page = key0 < kend ? bt[key0 >> p.page_shift] : -1;
         const int row = page >= 0 ? page * p.page_size + (key0 & (p.page_size - 1)) : 0;      // page 0 where there is none: cleared below
-        lf_tma_2d(base + b * STAGE_BYTES + chunk * LF_CHUNK + box * box_keys * 128, &kmap, chunk * 64, row, full(b));
+        const uint32_t dst = base + b * STAGE_BYTES + group * (NK * 1024) + chunk * 1024;
+        if (p.whole) lf_tma_3d(dst, &kmap, 0, row, 0, full(b));
+        else lf_tma_3d(dst, &kmap, chunk * 64, row, 0, full(b));
       }
     };
     // Vectors before the request's first token of this step were written by earlier steps: the first stages of them are requested while
@@ -172,7 +180,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
     if (kbase + LF_KEYS > kend || hole) {                    // uniform over the CTA
       const int first = hole ? 0 : kend - kbase;
       for (int idx = tid; idx < (LF_KEYS - first) * NK * 8; idx += LF_WARPS * 32)
-        asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(kb + lf_offset(LF_KEYS, first + idx / (NK * 8), idx % (NK * 8))), "r"(0) : "memory");
+        asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(kb + lf_stage_offset<NK>(first + idx / (NK * 8), idx % (NK * 8))), "r"(0) : "memory");
       lf_sync();
     }
 
@@ -188,7 +196,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
         ldmatrix_x4(q_smem + lf_offset(ROWS, a_row, kk * 2 + (lane >> 4)), a[0][0], a[0][1], a[0][2], a[0][3]);
         ldmatrix_x4(q_smem + lf_offset(ROWS, a_row, kk * 2 + 2 + (lane >> 4)), a[1][0], a[1][1], a[1][2], a[1][3]);
         // matrices: the four 16-byte pieces of two steps
-        ldmatrix_x4(kb + lf_offset(LF_KEYS, wn * KPW + (lane & 7), kk * 2 + (lane >> 3)), b0, b1, b2, b3);
+        ldmatrix_x4(kb + lf_stage_offset<NK>(wn * KPW + (lane & 7), kk * 2 + (lane >> 3)), b0, b1, b2, b3);
         mma_bf16(s[0], a[0], b0, b1);
         mma_bf16(s[0], a[1], b2, b3);
       }
@@ -201,7 +209,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
         for (int nb = 0; nb + 1 < NB; nb += 2) {
           // matrices: (keys nb, lo), (keys nb, hi), (keys nb + 1, lo), (keys nb + 1, hi)
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4(kb + lf_offset(LF_KEYS, wn * KPW + nb * 8 + (lane & 7) + (lane >> 4) * 8, kk * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
+          ldmatrix_x4(kb + lf_stage_offset<NK>(wn * KPW + nb * 8 + (lane & 7) + (lane >> 4) * 8, kk * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
           mma_bf16(s[nb], a, b0, b1);
           mma_bf16(s[nb + 1 < NB ? nb + 1 : nb], a, b2, b3);
         }
@@ -282,7 +290,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap kmap, LatentFlashParams 
       for (int db = 0; db < ND; db += 2) {
         // matrices (transposed on load): (keys lo, entries db), (keys hi, db), (keys lo, db + 1), (keys hi, db + 1)
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(kb + lf_offset(LF_KEYS, ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, v_col + db + (lane >> 4)), b0, b1, b2, b3);
+        ldmatrix_x4_trans(kb + lf_stage_offset<NK>(ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, v_col + db + (lane >> 4)), b0, b1, b2, b3);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma_bf16(o[mt][db], a[mt], b0, b1);
@@ -406,7 +414,7 @@ typedef CUresult (*LfEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, vo
                                const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 struct LfMapKey {
-  const void* base; long long rows; int d, box;
+  const void* base; long long rows; int d, box;             // box: chunks of a box
   bool operator==(const LfMapKey& o) const { return base == o.base && rows == o.rows && d == o.d && box == o.box; }
 };
 struct LfMapKeyHash {
@@ -419,7 +427,8 @@ struct LfMapKeyHash {
 static std::unordered_map<LfMapKey, CUtensorMap, LfMapKeyHash> g_lf_maps;
 static std::mutex g_lf_mu;
 
-// A pool [pages, page size, d] as rows of d entries: boxes of 64 entries x `box` rows; what lies past d reads as zeros.
+// A pool [pages, page size, d] as rows of d entries: boxes of 8 rows x 64 entries, and with chunks > 0 (d a multiple of 64) so many
+// chunks of 64 entries one behind the other; what lies past d reads as zeros.
 static bool lf_pool_map(CUtensorMap* out, const void* pool, long long rows, int d, int box) {
   LfMapKey key{pool, rows, d, box};
   std::lock_guard<std::mutex> g(g_lf_mu);
@@ -428,11 +437,11 @@ static bool lf_pool_map(CUtensorMap* out, const void* pool, long long rows, int 
   void* sym = nullptr;
   cudaDriverEntryPointQueryResult q;
   if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) return false;
-  cuuint64_t dims[2] = {(cuuint64_t)d, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)d * 2};
-  cuuint32_t bx[2] = {64, (cuuint32_t)box};
-  cuuint32_t estr[2] = {1, 1};
-  if (((LfEncodeFn)sym)(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(pool), dims, strides, bx, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+  cuuint64_t dims[3] = {(cuuint64_t)(box > 0 ? 64 : d), (cuuint64_t)rows, (cuuint64_t)(box > 0 ? d / 64 : 1)};
+  cuuint64_t strides[2] = {(cuuint64_t)d * 2, 128};
+  cuuint32_t bx[3] = {64, 8, (cuuint32_t)(box > 0 ? box : 1)};
+  cuuint32_t estr[3] = {1, 1, 1};
+  if (((LfEncodeFn)sym)(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(pool), dims, strides, bx, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return false;
   if (g_lf_maps.size() > 4096) g_lf_maps.clear();
@@ -489,27 +498,28 @@ LB_EXPORT int lb_latent_flash(const void* q, void* out, const void* pool, const 
   LB_CHECK_ARG(num_tiles <= 65535 && hgroups <= 65535, "latent_flash: too many tiles");
   if (num_tiles == 0) return 0;
   CUtensorMap map;
-  if (!lb::lf_pool_map(&map, pool, (long long)num_pages * page_size, dk, page_size < lb::LF_KEYS ? page_size : lb::LF_KEYS)) {
+  const int nk = (dk + 63) / 64, nv = (dv + 63) / 64;
+  const int nk_padded = nk <= 2 ? 2 : (nk <= 3 && nv <= 2) ? 3 : (nk <= 5 && nv <= 4) ? 5 : 9;
+  if (!lb::lf_pool_map(&map, pool, (long long)num_pages * page_size, dk, dk % 64 == 0 ? nk_padded : 0)) {
     lb::set_error("latent_flash: cuTensorMapEncodeTiled failed");
     return 3;
   }
   lb::LatentFlashParams p;
   p.q = (const lb::bf16*)q; p.out = (lb::bf16*)out; p.positions = positions; p.block_table = block_table; p.max_pages = max_pages;
   p.tiles = (const int4*)tiles; p.sinks = sinks; p.part_rows = part_rows; p.splits = splits; p.heads = heads; p.group = group;
-  p.dk = dk; p.dv = dv; p.page_size = page_size; p.scale_log2 = scale * 1.4426950408889634f;
+  p.dk = dk; p.dv = dv; p.page_size = page_size; p.scale_log2 = scale * 1.4426950408889634f; p.whole = dk % 64 == 0 ? 1 : 0;
   p.part_o = workspace;
   p.part_ml = splits > 1 ? workspace + (size_t)num_tiles * hgroups * splits * part_rows * dv : nullptr;
   p.page_shift = 0;
   while ((1 << p.page_shift) < page_size) ++p.page_shift;
-  const int nk = (dk + 63) / 64, nv = (dv + 63) / 64;
   const int mt = part_rows <= 16 ? 1 : (part_rows <= 32 ? 2 : 4);
   cudaError_t e;
 #define LB_LF(NK, NV) \
   (mt == 1 ? lb::lf_launch<NK, NV, 1>(map, p, num_tiles, hgroups, stream) : mt == 2 ? lb::lf_launch<NK, NV, 2>(map, p, num_tiles, hgroups, stream) \
                                                                                    : lb::lf_launch<NK, NV, 4>(map, p, num_tiles, hgroups, stream))
-  if (nk <= 2) e = LB_LF(2, 2);
-  else if (nk <= 3 && nv <= 2) e = LB_LF(3, 2);
-  else if (nk <= 5 && nv <= 4) e = LB_LF(5, 4);
+  if (nk_padded == 2) e = LB_LF(2, 2);
+  else if (nk_padded == 3) e = LB_LF(3, 2);
+  else if (nk_padded == 5) e = LB_LF(5, 4);
   else e = LB_LF(9, 8);
 #undef LB_LF
   if (e != cudaSuccess) { lb::set_error("latent_flash: cannot reserve shared memory: %s", cudaGetErrorString(e)); return 2; }

@@ -1398,8 +1398,8 @@ def latent_expansion_pays(tokens: int, span: int, heads: int, dim: int, rot: int
     than by the kernel that leaves them in latent space.  By the operations of both and the rates the kernels reach; it depends
     on the step's shape alone, so recordings keep it."""
     seen = span - 0.5 * tokens
-    expanded = 2.0 * span * heads * (dim + vdim) * kv_rank / 1.0e15 + 2.0 * (-(-tokens // 128) * 128) * seen * heads * (dim + rot + vdim) / 4.5e14 + 8e-6
-    absorbed = 2.0 * tokens * seen * heads * (2 * kv_rank + rot) / 2.2e14 + 2.0 * tokens * heads * kv_rank * (dim + vdim) / 2.5e14
+    expanded = 2.0 * span * heads * (dim + vdim) * kv_rank / 1.0e15 + 2.0 * (-(-tokens // 128) * 128) * seen * heads * (dim + rot + vdim) / 4.5e14 + 12e-6
+    absorbed = 2.0 * tokens * seen * heads * (2 * kv_rank + rot) / 1.4e14 + 2.0 * tokens * heads * kv_rank * (dim + vdim) / 2.5e14 + 20e-6
     return expanded < absorbed
 
 

@@ -41,7 +41,7 @@ from .linear import Linear
 # less than they gain: the padding is 64 places an expert on average, 127 at most, and the product several times faster.
 GROUPED_FROM = 96
 # Up to so many pairs an expert (on average) a step is a stream of the experts' weights and takes the kernel made for it, with row
-# tiles of 16 places (an expert with more reads its weights once a tile), or of 64 from FEW_UP_TO on.
+# tiles of 16 places (an expert with more reads its weights once a tile), or, for gated products, of 64 from FEW_UP_TO on.
 FEW_UP_TO, SOME_UP_TO = 8, 48
 
 
@@ -107,7 +107,7 @@ class ExpertBank(FeedForward):
             ops.expert_dispatch_padded(ids, E, pair_at, place_of, tile_group, rt.stream, tokens=tokens)
             return Dispatch(pair_at, place_of, tile_group=tile_group)
         offsets, pair_at = rt.empty((E + 1,), torch.int32), rt.empty((pairs,), torch.int32)
-        few = 0 if not self.grouped_ok else 1 if pairs <= FEW_UP_TO * E else 2 if pairs <= SOME_UP_TO * E else 0
+        few = 0 if not self.grouped_ok else 1 if pairs <= FEW_UP_TO * E else 2 if self.gated and pairs <= SOME_UP_TO * E else 0
         meta = rt.empty((4 + 3 * ops.expert_max_tiles(pairs, E, few),), torch.int32)
         ops.expert_dispatch(ids, E, offsets, pair_at, place_of, meta, rt.stream, tokens=tokens, few=few)
         return Dispatch(pair_at, place_of, meta=meta, few=few)
@@ -126,7 +126,7 @@ class ExpertBank(FeedForward):
             return y
         ops.expert_gemm(inner, h, self.gate_up, d.meta, d.pair_at, self.top, True, rt.stream, fast=rt.fast_kernels,
                         interleaved=self.interleaved, few=d.few, **how)
-        ops.expert_gemm(y, inner, self.down, d.meta, d.pair_at, self.top, False, rt.stream, fast=rt.fast_kernels, few=d.few)
+        ops.expert_gemm(y, inner, self.down, d.meta, d.pair_at, self.top, False, rt.stream, fast=rt.fast_kernels, few=d.few % 2)
         return y
 
 

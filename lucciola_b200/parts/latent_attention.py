@@ -148,10 +148,11 @@ class RotaryLatentAttention(Mixer):
         out = W_o concat_h( sigmoid(W_g u)_h * sum_j w_j v_h,j )
 
     [c | k_r] is all that is cached: one vector of kv_rank + rot_dim entries a token, key and value of one "head" whose values
-    are the first kv_rank entries (KVPages(1, kv_rank + rot_dim, shared=True)).  As in LatentAttention the head's key map
-    moves to the query and its value map behind the sum: attention runs as `heads` query heads [W_uk[h]^T q_u | q_r] over
-    the cached vectors.  W_q | W_dkv | W_g are one product with 32-bit output; one kernel norms the latent, rotates, and
-    writes the pages and the queries."""
+    are the first kv_rank entries (KVPages(1, kv_rank + rot_dim, shared=True)).  As in LatentAttention the head's key map moves
+    to the query and its value map behind the sum: attention runs as `heads` query heads [W_uk[h]^T q_u | q_r] over the cached
+    vectors (latent_flash.cu).  For longer portions that is several times the work of attention on the heads' own keys and
+    values, so these are multiplied out of the gathered latents first (latent_prefill.cu) where that pays.  W_q | W_dkv |
+    W_g are one product with 32-bit output; one kernel norms the latent, rotates, and writes the pages and the queries."""
     recordable = True
 
     def __init__(self, rt: Runtime, prefix: str, width: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int,

@@ -403,6 +403,7 @@ def test_padding_entries_of_a_recorded_step_read_nothing():
     pool[0] = pool[0].where(torch.tensor(bool((table == 0).any()), device=DEV), torch.tensor(float("nan"), device=DEV).to(torch.bfloat16))
     tiles = torch.tensor([(0, 1, 0, 0), (1, 1, 1, 0)], dtype=torch.int32, device=DEV)
     for splits in (1, 2):
+        out.fill_(float("nan"))
         ops.latent_flash(q, out, pool, step.positions, table, tiles, heads, heads, page, 0.1, splits, stream(), sinks=torch.zeros(heads, device=DEV))
         close(out[:1], want(0.1, torch.zeros(heads, device=DEV))[:1], torch.bfloat16)
         assert torch.isfinite(out).all()
